@@ -96,15 +96,20 @@ typedef enum ZgOpTag {
  * accumulation is f32.
  *
  * Control buffer `ctl` (int32 words inside an f32 buffer, written by the host before every execution):
- *   [0] position of the step's first token in its sequence, [1] state slot, [ZG_CTL_IDS ..) the step's token ids.
+ *   [0] position of the step's first token in its sequence, [1] state slot, [2] the sequence's token before the step (-1: the
+ *   step starts the sequence), [ZG_CTL_IDS ..) the step's token ids.
  *
  * EMBED             dst[t, :] = table[ids[t], :] * f0; with n3 = 1 a learned position row joins it, unscaled: + positions[p(t), :]
  *                   (a second table at off 1 of the same arena, p(t) = the token's position in its sequence)
- *                   buf 0 dst 1 ctl 2 table | off 0 table 1 positions | n 0 T 1 D 2 wdt 3 positions | f 0 scale
+ *                   with n4 > 0 a row of a bigram table joins it, unscaled: row (previous token * n5 + token * n6) mod n4, and row n4
+ *                   (the last of n4 + 1) for a sequence's first token (a third table at off 2; n5, n6 < n4; not together with n3)
+ *                   buf 0 dst 1 ctl 2 table | off 0 table 1 positions 2 bigram | n 0 T 1 D 2 wdt 3 positions 4 bigram buckets
+ *                   5 factor of the previous token 6 factor of the token | f 0 scale
  * LINEAR            dst[m, n] = act(sum_k src[m, k] W[n, k] (+ bias[n])); act (n6): 0 none, 1 + the ACTIVATION kind otherwise (f0: its
- *                   parameter, where the kind has one)
+ *                   parameter, where the kind has one), on the columns [n8, n9) alone (n9 = 0: up to N): a stacked projection whose
+ *                   parts differ
  *                   buf 0 dst 1 src 2 W 3 bias 4 ctl | off 0 W 1 bias 2 src 3 dst | n 0 M 1 N 2 K 3 src row stride 4 dst row stride 5 wdt 6 act
- *                   7 source slot stride
+ *                   7 source slot stride 8 first column of act 9 end of its columns
  *                   With n7 > 0 the source rows are those of a per-sequence state buffer (a ring): n7 elements per slot, the slot
  *                   from the control buffer buf 4.
  *                   f 0 activation parameter
@@ -115,17 +120,20 @@ typedef enum ZgOpTag {
  *                   (cols values) and the scalar alpha follow w in its arena; kind bit 4: no norm and no weight, the row
  *                   itself (times the gain with bit 2): dst = res + gain * src, the plain residual step of a pre-norm stack.
  *                   Bits 3 and 4 combine with a residual and a chained norm, not with the averaged source or the token shift.
+ *                   kind bit 5 (kinds with statistics): the weight is a single number for all columns
  *                   with n7 = 1 (kinds with statistics, no averaged source): buf 6 is a SECOND source, normed like the first with a
  *                   weight of its own (off 2 of w's arena) and added to it: dst = res + norm(src) w + norm(src2) w_b
+ *                   with n8 = 1 + kind (kinds with statistics): the normed source, or the sum of the two, passes another norm (weight at
+ *                   off 5 of w's arena) before it joins the residual: dst = res + norm_o(norm(src) w + norm(src2) w_b) w_o
  *                   with buf 4: also dst2 = norm(dst) * w2 in the same launch (the norm closing a sublayer and the one opening the next)
  *                   with buf 6 (single-row steps): the last output of the launch then passes a TOKEN_SHIFT (mix at off 2 of the
  *                   arena of the norm it follows, state buf 6, ctl buf 7) in the same launch
  *                   w and w2 must be constants of the model (an uploaded arena): they are read before the producing op of src has finished
  *                   with n 5 > 0 (no res, no chained norm): the row that is normed is the DEPTH_MIX of n5 streams of src (stride n6,
  *                   coefficients at off 4 of w's arena); buf 4 receives that average itself
- *                   buf 0 dst 1 src 2 w 3 res 4 dst2 5 w2 6 shift state 7 ctl | off 0 w 1 w2 2 shift mix 3 dst 4 average coefficients
+ *                   buf 0 dst 1 src 2 w 3 res 4 dst2 5 w2 6 shift state 7 ctl | off 0 w 1 w2 2 shift mix 3 dst 4 average coefficients 5 outer norm
  *                   n 0 rows 1 cols 2 kind 3 wdt 5 averaged streams 6 their stride 7 second source
- *                   4 kind of dst2 | f 0 eps 1 gain
+ *                   4 kind of dst2 8 outer norm | f 0 eps 1 gain
  * WINDOW_ATTENTION  causal attention over the last `window` positions whose keys double as values (one projection, one cache),
  *                   grouped query heads, scores capped smoothly (cap * tanh(s / cap), f1 = 0: off), a per-distance per-head
  *                   additive bias table [window, H] (f32 program buffer), a softmax whose denominator carries an extra 1 (a
@@ -150,13 +158,14 @@ typedef enum ZgOpTag {
  *                   off 0 q 1 k 2 v (columns of a qkv row) 3 beta (column of its row) 4 A_log 5 dt_bias 6 norm_w (weights)
  *                   7 gate (column of its row)
  *                   n 0 T 1 H 2 G 3 dim 4 vdim 5 qkv row stride 6 beta row stride 7 a row stride 8 gate row stride 9 wdt
- *                   10 form 11 dst row stride (0: H * vdim) 12 dst column
+ *                   10 form 11 dst row stride (0: H * vdim) 12 dst column 13 a (column of its row)
  *                   f 0 output-norm eps 1 unit-vector eps 2 q scale 3 decay temperature 4 output scale
  *                   Form bits (n10), all clear for the rule above.  Bit 0, plain accumulation (gated linear attention): no
  *                   unit vectors (q is only scaled by f2) and no correction by what the state already holds, u = v:
  *                   S <- g * S + k v^T, o = S^T q; buf 2 is not read.  Bit 1: the decay is g = sigmoid(a + dt_bias)^(1 / f3),
  *                   evaluated as exp(-softplus(-(a + dt_bias)) / f3); A_log is not read.  Bit 2: the output gate is
- *                   silu(gate) instead of sigmoid(gate).  Bit 3: the result is multiplied by f4.  It may land in columns of a
+ *                   silu(gate) instead of sigmoid(gate).  Bit 4: one decay per head instead of one per key channel (a row of buf 3 and
+ *                   dt_bias hold H values).  Bit 3: the result is multiplied by f4.  It may land in columns of a
  *                   wider row (n11, n12), beside another mixer's heads.
  * ROUTE             mode 0: s = softmax(logits) over all NE outputs; the `top` largest of s + correction are chosen (ties:
  *                   lowest index); dst[t, c] = {index as int32 bits, s[index]} (weights not renormalised)
@@ -193,16 +202,23 @@ typedef enum ZgOpTag {
  *                   With n10 > 0 (and n9 > 0) every normed group — key heads, and the query heads of off5 — is first turned by
  *                   the token's rotary position on its first n10 values (layout n8; frequencies base^(-2i / n10) from f1, or
  *                   from the f32 table buf 4 at element off 7, as ROTARY takes it), and the root mean square is that of the
- *                   turned vector: ROTARY fused, for designs that norm after the rotation.
- *                   buf 0 cache 1 src 2 ctl 3 norm weight 4 frequency table | off 0 src column 1 cache column 2 norm weight 3 query column
+ *                   turned vector: ROTARY fused, for designs that norm after the rotation.  n13 = 1: norm and weight come first and
+ *                   the normed vector is turned; n13 = 2: the heads are turned and not normed (no weight is read).
+ *                   With n11 > 0 the launch also keeps POOLED BLOCKS: row b of buf 5 (external [slots, n12, width]) becomes the mean of
+ *                   the cached rows of positions b n11 .. b n11 + n11 - 1.  A step from position p leaves the blocks whose last
+ *                   position is p - 1 .. p + T - 2 (a block is asked for at the earliest one position after its last).
+ *                   buf 0 cache 1 src 2 ctl 3 norm weight 4 frequency table 5 pooled rows | off 0 src column 1 cache column 2 norm weight 3 query column
  *                   4 query weight 5 query heads 6 temperature period 7 frequency table offset
  *                   n 0 T 1 columns 2 src row stride 3 width 4 R 5 normed 6 rot 7 wdt 8 rotary layout 9 norm group 10 rotary inside the groups
+ *                   11 positions per pooled block 12 pooled rows 13 order of norm and rotation
  *                   f 0 eps 1 rotary base 2 temperature coefficient
  * CACHED_ATTENTION  softmax attention of the step's queries over cached keys and values.  A query row holds H * maps vectors
  *                   of dk (head h, map m at (h * maps + m) * dk); a key row G * maps vectors of dk; a value row G vectors of
  *                   dv; query (h, m) reads key (h / (H / G), m) and value h / (H / G).  The value cache may be the key cache
  *                   (a latent that serves as both).  Masks: 0 causal, 1 the last `size` positions, 2 causal inside blocks
- *                   of `size` positions counted from position 0.  R must cover what the mask can reach plus the step.
+ *                   of `size` positions counted from position 0, 3 the last `size` positions and, as one key and value each, the pooled
+ *                   blocks (CACHE_APPEND) of n15 positions that lie wholly before them: rows of buf 7 (external [slots, off 6, key row
+ *                   width], the layout of the one cache that holds keys and values; no score table with this mask).  R must cover what the mask can reach plus the step.
  *                   With buf 5 a score table [H * maps, off 6] (f32) indexed by the distance i - j is added to the scaled score
  *                   (any distance bias; a constant per head folds into it).  Weights (off 5): 0 softmax over the visible keys,
  *                   1 sigmoid(score) of every visible key, not normalised over the keys.
@@ -212,12 +228,12 @@ typedef enum ZgOpTag {
  *                   neither scaled nor capped, and counts once (a weight operand: element off 7 of buf 6, type n12).  The
  *                   result is multiplied by f2 where n13 = 1 and may land in columns of a wider row (n10 row stride, 0: H * maps * dv;
  *                   n11 first column), beside another mixer's heads.
- *                   buf 0 dst [T, H * maps, dv] 1 q 2 key cache 3 value cache 4 ctl 5 score table 6 sinks
- *                   off 0 q column 1 key column 2 value column (inside a cache row) 3 mask kind 4 mask size 5 weights 6 table row length
+ *                   buf 0 dst [T, H * maps, dv] 1 q 2 key cache 3 value cache 4 ctl 5 score table 6 sinks 7 pooled rows
+ *                   off 0 q column 1 key column 2 value column (inside a cache row) 3 mask kind 4 mask size 5 weights 6 table row length (mask 3: pooled rows)
  *                   7 sinks
  *                   n 0 T 1 H 2 G 3 maps 4 dk 5 dv 6 q row stride 7 key row width 8 value row width 9 R 10 dst row stride
  *                   11 dst column 12 wdt of the sinks 13 output scale given 14 caches without slots (rows the program itself computed
- *                   for this step, position p in row p mod R as in a ring) | f 0 score scale 1 score cap 2 output scale
+ *                   for this step, position p in row p mod R as in a ring) 15 positions per pooled block | f 0 score scale 1 score cap 2 output scale
  * MAP_COMBINE       differential attention's combination of two maps: o = a[.., 0, :] - f0 * a[.., 1, :], then
  *                   o / sqrt(mean(o^2) + f1) * f2 per (token, head)
  *                   buf 0 dst [rows, dv] 1 src [rows, 2, dv] | n 0 rows 1 dv | f 0 lambda 1 eps 2 output scale
@@ -231,27 +247,30 @@ typedef enum ZgOpTag {
  *                   element by element, (a, b, c, e) four weights; may run in place
  *                   buf 0 dst 1 src 2 coefficients | off 0 coefficients | n 0 T 1 columns 2 wdt | f 0 eps
  * SSM_SCAN          state-space recurrence with one scalar decay per head and token (Mamba-2): dt = softplus(dt_logit + dt_bias[h]),
- *                   S <- exp(-exp(A_log[h]) dt) S + dt B x^T (S is N x P per head, f32), y = S^T C + D[h] x.  Head h reads the B and
+ *                   S <- exp(-exp(A_log[h]) dt) S + dt B x^T (S is N x P per head, f32), y = S^T C + D[h] x.  With n8 = 1 (lightning
+ *                   attention: B, C and x are keys, queries and values) the decay is a constant per head, the step size 1 and there is
+ *                   no D x: S <- g[h] S + B x^T, y = S^T C, g an f32 table in buf 2 at off 3.  Head h reads the B and
  *                   C of group h / (H / G).  x | B | C are columns of one row (the output of the short convolution), the dt
  *                   logits columns of another.  The state is external [slots, zg_cuda_seq_state_elems(op)] in a layout private
  *                   to the op, zeros for a fresh slot.
  *                   buf 0 dst [T, H * P] 1 xbc 2 dt 3 weights 4 state 5 ctl
  *                   off 0 x 1 B 2 C (columns of an xbc row) 3 dt (column of its row) 4 A_log 5 dt_bias 6 D (weights)
- *                   n 0 T 1 H 2 G 3 N 4 P 5 xbc row stride 6 dt row stride 7 wdt
+ *                   n 0 T 1 H 2 G 3 N 4 P 5 xbc row stride 6 dt row stride 7 wdt 8 constant decays
  * MIN_GRU           gated recurrence whose gates read the current token only: z = sigmoid(zl), c = u + 1/2 where u >= 0 and
  *                   sigmoid(u) where u < 0, S <- (1 - z) S + z c element by element (external [slots, W], zeros for a fresh
  *                   slot), dst = S * silu(g).  zl | u | g are columns of one row (biases belong to the projection).
  *                   buf 0 dst 1 proj 2 state 3 ctl | off 0 zl 1 u 2 g (columns) | n 0 T 1 W 2 proj row stride 3 dst row stride
  * GATED_NORM        dst = N(src * silu(gate)) * w with N an RMS norm over each of n2 equal parts of the row (the gate comes
- *                   before the norm); may run in place
+ *                   before the norm); may run in place.  n7 bit 0: the gate comes after, N(src) * w * gate; bit 1: sigmoid(gate)
+ *                   instead of silu(gate)
  *                   buf 0 dst 1 src 2 gate 3 w | off 0 gate column 1 w | n 0 T 1 columns 2 groups 3 gate row stride 4 wdt
- *                   5 src row stride 6 dst row stride | f 0 eps
+ *                   5 src row stride 6 dst row stride 7 form | f 0 eps
  * HEAD_NORM         per-head RMS norm in place with one weight of `dim` values shared by the heads, times a temperature that
  *                   grows with the position p of the token: 1 + f1 * ln(floor((p + 1) / n5) + 1) (n5 = 0: none)
  *                   buf 0 x 1 w 2 ctl | off 0 column of the first head 1 w | n 0 T 1 heads 2 dim 3 row stride 4 wdt 5 period
  *                   f 0 eps 1 temperature coefficient
  * ACTIVATION        dst = act(src) element by element, may run in place; kinds: 0 relu(z)^2, 1 silu, 2 gelu (tanh form), 3 relu,
- *                   4 smooth cap f0 * tanh(z / f0)
+ *                   4 smooth cap f0 * tanh(z / f0), 5 gelu (erf form)
  *                   buf 0 dst 1 src | n 0 elements 1 kind | f 0 parameter of the kind
  * RG_LRU            real-gated linear recurrent unit, element by element over W channels: r = sigmoid(rl + r_bias),
  *                   i = sigmoid(il + i_bias), log a = -f0 * r * softplus(lam), S <- a S + sqrt(1 - a^2) (i u) (external
@@ -267,6 +286,7 @@ typedef enum ZgOpTag {
 #define ZG_W_BF16 1
 #define ZG_CTL_POS 0
 #define ZG_CTL_SLOT 1
+#define ZG_CTL_PREV 2
 #define ZG_CTL_IDS 8
 typedef struct ZgSeqOp {
     uint32_t buf[8];

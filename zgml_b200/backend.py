@@ -207,34 +207,45 @@ class DeviceOp:
         return o
 
     @staticmethod
-    def embed(dst, ctl, table, table_off, T, D, scale, wdt, positions_off=None):
-        """Rows of the table times `scale`; with `positions_off` a learned position row of the same arena is added, unscaled."""
-        return DeviceOp._seq(abi.OP_EMBED, [dst, ctl, table], [table_off, positions_off or 0], [T, D, wdt, int(positions_off is not None)], [scale])
+    def embed(dst, ctl, table, table_off, T, D, scale, wdt, positions_off=None, bigram=None):
+        """Rows of the table times `scale`; with `positions_off` a learned position row of the same arena is added, unscaled.
+        `bigram` = (offset, buckets, mul_prev, mul_cur): a row of that table (buckets + 1 rows in the same arena) is added, unscaled, at
+        (previous token * mul_prev + token * mul_cur) mod buckets; a sequence's first token takes the last row."""
+        b_off, buckets, mul_prev, mul_cur = bigram or (0, 0, 0, 0)
+        if buckets:
+            mul_prev, mul_cur = mul_prev % buckets, mul_cur % buckets       # the same residues, and the products fit the kernel's integers
+        return DeviceOp._seq(abi.OP_EMBED, [dst, ctl, table], [table_off, positions_off or 0, b_off], [T, D, wdt, int(positions_off is not None), buckets, mul_prev, mul_cur], [scale])
 
     @staticmethod
-    def linear(dst, src, w, w_off, M, N, K, wdt, bias=None, bias_off=0, src_off=0, dst_off=0, src_rs=0, dst_rs=0, act=None, act_param=0.0, ctl=None, src_slot_stride=0):
-        """`act`: an activation of abi.ACTIVATIONS applied in the epilogue, after the bias (`act_param`: its parameter, where it has one).
+    def linear(dst, src, w, w_off, M, N, K, wdt, bias=None, bias_off=0, src_off=0, dst_off=0, src_rs=0, dst_rs=0, act=None, act_param=0.0, ctl=None, src_slot_stride=0,
+               act_cols=None):
+        """`act`: an activation of abi.ACTIVATIONS applied in the epilogue, after the bias (`act_param`: its parameter, where it has one), to
+        the output columns act_cols = (first, end) only, where given.
         `src_slot_stride` > 0: the source rows are the slot's part of a per-sequence state buffer (that many elements per slot; slot from `ctl`)."""
         return DeviceOp._seq(abi.OP_LINEAR, [dst, src, w, bias, ctl if src_slot_stride else None], [w_off, bias_off, src_off, dst_off],
-                             [M, N, K, src_rs or K, dst_rs or N, wdt, 0 if act is None else abi.ACTIVATIONS[act] + 1, src_slot_stride], [act_param])
+                             [M, N, K, src_rs or K, dst_rs or N, wdt, 0 if act is None else abi.ACTIVATIONS[act] + 1, src_slot_stride] + list(act_cols or ()), [act_param])
 
     @staticmethod
     def norm(dst, src, w, w_off, rows, cols, eps, wdt, kind="layer", res=None, then=None, then_w=None, then_w_off=0, then_kind="layer",
-             gain=None, shift_state=None, shift_off=0, ctl=None, dst_off=0, average=None, src2=None, src2_w_off=0):
+             gain=None, shift_state=None, shift_off=0, ctl=None, dst_off=0, average=None, src2=None, src2_w_off=0,
+             outer=None, outer_w_off=0):
         """dst = (res +) norm(src; w); with `then`, also then = norm(dst; weights at then_w_off of arena then_w) in the same launch.
-        Kinds: "layer", "rms", and "rms1" (RMS norm whose weight is stored around zero, applied as 1 + w).  `gain` multiplies the
+        Kinds: "layer", "rms", "rms1" (RMS norm whose weight is stored around zero, applied as 1 + w) and "rms_scalar" (RMS norm whose weight is
+        one number).  `outer`: a kind; what the source(s) gave passes that norm too (weight at outer_w_off of arena w) before the residual.  `gain` multiplies the
         result(s); `shift_state` (single-row steps, with `then`) passes `then` through a token shift whose mix lies at shift_off of
         then_w (of w without `then`) and whose carried row is that state buffer.  `average` = (out, coeff_off, terms, stride): the
         row that is normed is sum_j coeff[j] * src[j * stride + .] (coefficients in w's arena), which also goes to buffer `out`."""
-        kinds = {"layer": abi.NORM_LAYER, "rms": abi.NORM_RMS, "rms1": abi.NORM_RMS | abi.NORM_UNIT_OFFSET,
+        kinds = {"layer": abi.NORM_LAYER, "rms": abi.NORM_RMS, "rms1": abi.NORM_RMS | abi.NORM_UNIT_OFFSET, "rms_scalar": abi.NORM_RMS | abi.NORM_SCALAR_WEIGHT,
                  "dyt": abi.NORM_DYNAMIC_TANH, "none": abi.NORM_NONE}
         if src2 is not None:
             # Two sources, each normed with a weight of its own (both in arena w) and added: dst = res + gain (norm(src) w + norm(src2) w2).
-            assert kind in ("layer", "rms", "rms1") and average is None and shift_state is None
+            assert kind in ("layer", "rms", "rms1", "rms_scalar") and average is None and shift_state is None
             g1 = abi.NORM_GAIN if gain is not None else 0
             return DeviceOp._seq(abi.OP_NORM, [dst, src, w, res, then, then_w if then is not None and then_kind != "none" else None, src2],
-                                 [w_off, then_w_off, src2_w_off, dst_off], [rows, cols, kinds[kind] | g1, wdt, kinds[then_kind] if then is not None else 0, 0, 0, 1],
+                                 [w_off, then_w_off, src2_w_off, dst_off, 0, outer_w_off],
+                                 [rows, cols, kinds[kind] | g1, wdt, kinds[then_kind] if then is not None else 0, 0, 0, 1, 0 if outer is None else 1 + kinds[outer]],
                                  [eps, gain if gain is not None else 0.0])
+        assert outer is None or (kind not in ("dyt", "none") and gain is None and average is None and shift_state is None)
         if kind in ("dyt", "none") or (then is not None and then_kind in ("dyt", "none")):
             # Kinds without row statistics: "dyt" = tanh(alpha x) w + b (bias and alpha follow w in its arena), "none" = the row itself.
             # The gain belongs to the FIRST norm here (dst = res + gain * f(src), the residual step of a pre-norm stack).
@@ -251,8 +262,8 @@ class DeviceOp:
             return DeviceOp._seq(abi.OP_NORM, [dst, src, w, None, then, None, shift_state, ctl if fused else None], [w_off, 0, shift_off, dst_off, avg_off],
                                  [rows, cols, kinds[kind] | g, wdt, 0, avg_terms, avg_stride], [eps, gain if gain is not None else 0.0])
         return DeviceOp._seq(abi.OP_NORM, [dst, src, w, res, then, then_w if then is not None else None, shift_state, ctl if fused else None],
-                             [w_off, then_w_off, shift_off, dst_off],
-                             [rows, cols, kinds[kind] | (g if then is None else 0), wdt, kinds[then_kind] | (g if then is not None else 0)],
+                             [w_off, then_w_off, shift_off, dst_off, 0, outer_w_off],
+                             [rows, cols, kinds[kind] | (g if then is None else 0), wdt, kinds[then_kind] | (g if then is not None else 0), 0, 0, 0, 0 if outer is None else 1 + kinds[outer]],
                              [eps, gain if gain is not None else 0.0])
 
     @staticmethod
@@ -268,16 +279,16 @@ class DeviceOp:
     @staticmethod
     def delta_rule(dst, qkv, beta, a, gate, w, state, ctl, q_off, k_off, v_off, beta_off, a_log_off, dt_bias_off, norm_off,
                    T, H, G, dim, vdim, qkv_rs, beta_rs, a_rs, gate_rs, wdt, norm_eps, unit_eps, q_scale, gate_off=0, plain=False, decay_tau=None,
-                   silu_gate=False, out_scale=None, dst_rs=0, dst_col=0):
+                   silu_gate=False, out_scale=None, dst_rs=0, dst_col=0, head_decay=False, a_col=0):
         """`plain`: no unit vectors and no correction by the state (S <- g S + k v^T: gated linear attention; `beta` may be None).
         `decay_tau`: the decay is sigmoid(a + dt_bias)^(1 / tau) instead of exp(-exp(A_log) softplus(a + dt_bias)).  `silu_gate`: the
-        output gate is silu instead of sigmoid.  `out_scale` multiplies the result, which may land at column `dst_col` of rows
+        output gate is silu instead of sigmoid.  `head_decay`: one decay per head (rows of `a` and dt_bias hold H values).  `out_scale` multiplies the result, which may land at column `dst_col` of rows
         `dst_rs` wide."""
         form = (abi.DELTA_PLAIN if plain else 0) | (abi.DELTA_SIGMOID_DECAY if decay_tau is not None else 0) | (abi.DELTA_SILU_GATE if silu_gate else 0) | \
-            (abi.DELTA_OUT_SCALE if out_scale is not None else 0)
+            (abi.DELTA_OUT_SCALE if out_scale is not None else 0) | (abi.DELTA_HEAD_DECAY if head_decay else 0)
         return DeviceOp._seq(abi.OP_DELTA_RULE, [dst, qkv, beta, a, gate, w, state, ctl],
                              [q_off, k_off, v_off, beta_off, a_log_off, dt_bias_off, norm_off, gate_off],
-                             [T, H, G, dim, vdim, qkv_rs, beta_rs, a_rs, gate_rs, wdt, form, dst_rs, dst_col], [norm_eps, unit_eps, q_scale, decay_tau or 0.0, out_scale or 0.0])
+                             [T, H, G, dim, vdim, qkv_rs, beta_rs, a_rs, gate_rs, wdt, form, dst_rs, dst_col, a_col], [norm_eps, unit_eps, q_scale, decay_tau or 0.0, out_scale or 0.0])
 
     @staticmethod
     def route(dst, logits, w, corr_off, T, n_outputs, top, wdt, logits_off=0, logits_rs=0, mode="corrected_softmax", groups=0, groups_kept=0):
@@ -311,28 +322,35 @@ class DeviceOp:
     @staticmethod
     def cache_append(cache, src, ctl, src_col, cache_col, T, cols, src_rs, width, rows, norm_w=None, norm_off=0, normed=0, eps=0.0, wdt=0,
                      rot=0, rot_base=0.0, rot_layout="pairs", norm_group=0, q_heads=0, q_col=0, q_norm_off=0, temp_coef=0.0, temp_every=0, head_rot=0,
-                     freqs=None, freqs_off=0):
+                     freqs=None, freqs_off=0, order="rotate_norm", pooled=None, pool=0, pool_rows=0):
         """`norm_group` > 0: the normed columns are normed in groups of that many (key heads) sharing one weight of that size.
         `q_heads` > 0: that many query heads of norm_group values at column q_col of the source rows are normed in place by the same
         launch (weight at q_norm_off of norm_w's arena), times the position-dependent temperature of HEAD_NORM.
         `head_rot` > 0: every normed group (key and query heads) is first turned by the token's rotary position on its first head_rot
-        values (`rot_layout`; frequencies from `rot_base`, or from the f32 table `freqs` at element `freqs_off`), then normed."""
-        return DeviceOp._seq(abi.OP_CACHE_APPEND, [cache, src, ctl, norm_w if normed else None, freqs if head_rot else None],
+        values (`rot_layout`; frequencies from `rot_base`, or from the f32 table `freqs` at element `freqs_off`), then normed;
+        `order` "norm_rotate": normed and weighted first, then turned; "rotate": turned and not normed (norm_w may be None).
+        `pool` > 0: row b of `pooled` (`pool_rows` rows per slot) becomes the mean of the cached rows of block b of `pool` positions."""
+        orders = {"rotate_norm": abi.ROTATE_THEN_NORM, "norm_rotate": abi.NORM_THEN_ROTATE, "rotate": abi.ROTATE_ONLY}
+        return DeviceOp._seq(abi.OP_CACHE_APPEND, [cache, src, ctl, norm_w if normed else None, freqs if head_rot else None, pooled if pool else None],
                              [src_col, cache_col, norm_off, q_col, q_norm_off, q_heads, temp_every, freqs_off],
-                             [T, cols, src_rs, width, rows, normed, rot, wdt, {"pairs": 0, "halves": 1}[rot_layout], norm_group, head_rot], [eps, rot_base, temp_coef])
+                             [T, cols, src_rs, width, rows, normed, rot, wdt, {"pairs": 0, "halves": 1}[rot_layout], norm_group, head_rot, pool, pool_rows, orders[order]],
+                             [eps, rot_base, temp_coef])
 
     @staticmethod
     def cached_attention(dst, q, k_cache, v_cache, ctl, q_col, k_col, v_col, T, H, G, maps, dk, dv, q_rs, k_width, v_width, rows, scale,
                          mask="causal", mask_size=0, weights="softmax", score_table=None, table_len=0, softcap=0.0, sink=None, sink_off=0, sink_wdt=0,
-                         out_scale=None, dst_rs=0, dst_col=0, unslotted=False):
+                         out_scale=None, dst_rs=0, dst_col=0, unslotted=False, pooled=None, pool=0, pool_rows=0):
         """`unslotted`: the caches are rows the program computed for this step (no state slots).  `score_table`: an f32 buffer [H * maps, table_len] added to the scaled scores by distance; `weights` "sigmoid": every
         visible key weighs sigmoid(score), not normalised over the keys.  `softcap` > 0: the scaled score passes cap * tanh(s / cap).
         `sink`: a weight buffer with one learned score per (head, map) at `sink_off` whose exponential joins the softmax's denominator.
-        `out_scale` multiplies the result, which may land at column `dst_col` of rows `dst_rs` wide."""
-        kinds = {"causal": abi.MASK_CAUSAL, "window": abi.MASK_WINDOW, "block": abi.MASK_BLOCK}
-        return DeviceOp._seq(abi.OP_CACHED_ATTENTION, [dst, q, k_cache, v_cache, ctl, score_table, sink],
-                             [q_col, k_col, v_col, kinds[mask], mask_size, {"softmax": abi.WEIGHTS_SOFTMAX, "sigmoid": abi.WEIGHTS_SIGMOID}[weights], table_len, sink_off],
-                             [T, H, G, maps, dk, dv, q_rs, k_width, v_width, rows, dst_rs, dst_col, sink_wdt, int(out_scale is not None), int(unslotted)], [scale, softcap, out_scale or 0.0])
+        `out_scale` multiplies the result, which may land at column `dst_col` of rows `dst_rs` wide.  Mask "pooled": the last mask_size positions
+        and the rows of `pooled` (`pool_rows` per slot, kept by CACHE_APPEND) whose blocks of `pool` positions lie wholly before them."""
+        kinds = {"causal": abi.MASK_CAUSAL, "window": abi.MASK_WINDOW, "block": abi.MASK_BLOCK, "pooled": abi.MASK_POOLED}
+        assert mask != "pooled" or score_table is None
+        return DeviceOp._seq(abi.OP_CACHED_ATTENTION, [dst, q, k_cache, v_cache, ctl, score_table, sink, pooled if mask == "pooled" else None],
+                             [q_col, k_col, v_col, kinds[mask], mask_size, {"softmax": abi.WEIGHTS_SOFTMAX, "sigmoid": abi.WEIGHTS_SIGMOID}[weights], pool_rows if mask == "pooled" else table_len, sink_off],
+                             [T, H, G, maps, dk, dv, q_rs, k_width, v_width, rows, dst_rs, dst_col, sink_wdt, int(out_scale is not None), int(unslotted),
+                              pool if mask == "pooled" else 0], [scale, softcap, out_scale or 0.0])
 
     @staticmethod
     def map_combine(dst, src, rows, dv, lam, eps, out_scale):
@@ -353,17 +371,21 @@ class DeviceOp:
         return DeviceOp._seq(abi.OP_POLY_NORM, [dst, src, w], [coeff_off], [T, cols, wdt], [eps])
 
     @staticmethod
-    def ssm_scan(dst, xbc, dt, w, state, ctl, x_col, b_col, c_col, dt_col, a_log_off, dt_bias_off, d_off, T, H, G, N, P, xbc_rs, dt_rs, wdt):
+    def ssm_scan(dst, xbc, dt, w, state, ctl, x_col, b_col, c_col, dt_col, a_log_off, dt_bias_off, d_off, T, H, G, N, P, xbc_rs, dt_rs, wdt, constant_decay=False):
+        """`constant_decay`: S <- g[h] S + B x^T, y = S^T C (lightning attention); `dt` is an f32 table with the heads' decays at dt_col, and `w`
+        and its offsets are not read."""
         return DeviceOp._seq(abi.OP_SSM_SCAN, [dst, xbc, dt, w, state, ctl], [x_col, b_col, c_col, dt_col, a_log_off, dt_bias_off, d_off],
-                             [T, H, G, N, P, xbc_rs, dt_rs, wdt])
+                             [T, H, G, N, P, xbc_rs, dt_rs, wdt, int(constant_decay)])
 
     @staticmethod
     def min_gru(dst, proj, state, ctl, z_col, u_col, g_col, T, W, proj_rs, dst_rs=0):
         return DeviceOp._seq(abi.OP_MIN_GRU, [dst, proj, state, ctl], [z_col, u_col, g_col], [T, W, proj_rs, dst_rs or W])
 
     @staticmethod
-    def gated_norm(dst, src, gate, w, w_off, gate_col, T, cols, groups, gate_rs, eps, wdt, src_rs=0, dst_rs=0):
-        return DeviceOp._seq(abi.OP_GATED_NORM, [dst, src, gate, w], [gate_col, w_off], [T, cols, groups, gate_rs, wdt, src_rs or cols, dst_rs or cols], [eps])
+    def gated_norm(dst, src, gate, w, w_off, gate_col, T, cols, groups, gate_rs, eps, wdt, src_rs=0, dst_rs=0, gate_after=False, sigmoid_gate=False):
+        """norm(src * silu(gate)) w in `groups` equal parts; `gate_after`: norm(src) w * silu(gate); `sigmoid_gate`: sigmoid instead of silu."""
+        form = (abi.GATE_AFTER if gate_after else 0) | (abi.GATE_SIGMOID if sigmoid_gate else 0)
+        return DeviceOp._seq(abi.OP_GATED_NORM, [dst, src, gate, w], [gate_col, w_off], [T, cols, groups, gate_rs, wdt, src_rs or cols, dst_rs or cols, form], [eps])
 
     @staticmethod
     def head_norm(x, w, w_off, ctl, col, T, heads, dim, row_stride, eps, wdt, temp_coef=0.0, temp_every=0):

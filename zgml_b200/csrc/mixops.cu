@@ -64,14 +64,41 @@ __global__ void k_rotary(float* x, const float* src, const float* __restrict__ c
 }
 
 // ── CACHE_APPEND: one CTA per token ──────────────────────────────────────────────────────────────────────────────
+// Pooled blocks: block b is the mean of the cached rows of positions b P .. b P + P - 1.  A step of T tokens from position p leaves
+// the blocks that ended at p - 1 .. p + T - 2: whoever attends over them sees a block at the earliest from the position after its
+// last one, so a single-token step averages nothing but rows of earlier steps and needs no launch of its own.
+// The i-th of a step's blocks; columns first, first + stride, ...
+__device__ void pool_block(float* __restrict__ pooled, const float* __restrict__ cache, const float* __restrict__ ctl, uint32_t T, uint32_t cols, uint32_t width, uint32_t R,
+                           uint32_t P, uint32_t pool_rows, uint32_t i, uint32_t first, uint32_t stride) {
+    const uint32_t p0 = (uint32_t)ctl_word(ctl, ZG_CTL_POS), slot = (uint32_t)ctl_word(ctl, ZG_CTL_SLOT);
+    const uint32_t end = (p0 + P - 1) / P + i;         // blocks up to and including this one
+    if (end == 0 || end > pool_rows || end * P > p0 + T - 1) return;
+    const float* rows = cache + (size_t)slot * R * width;
+    float* out = pooled + ((size_t)slot * pool_rows + end - 1) * width;
+    for (uint32_t c = first; c < cols; c += stride) {
+        float sum = 0.0f;
+#pragma unroll 4
+        for (uint32_t r = 0; r < P; r++) sum += rows[(size_t)(((end - 1) * P + r) % R) * width + c];
+        out[c] = sum / (float)P;
+    }
+}
+__global__ void k_block_pool(float* __restrict__ pooled, const float* __restrict__ cache, const float* __restrict__ ctl, uint32_t T, uint32_t cols, uint32_t width, uint32_t R, uint32_t P,
+                             uint32_t pool_rows) {
+    pdl_enter();
+    pool_block(pooled, cache, ctl, T, cols, width, R, P, pool_rows, blockIdx.x, blockIdx.y * blockDim.x + threadIdx.x, gridDim.y * blockDim.x);
+}
 // A cache row is [normed | rotated | plain]: the first `normed` columns are divided by their root mean square and weighted
 // (a latent), the next `rot` columns get the token's rotary position (a key part shared by the heads), the rest is copied.
 template <typename WT>
 __global__ void k_cache_append(float* __restrict__ cache, const float* __restrict__ src, const float* __restrict__ ctl, const WT* __restrict__ nw_,
                                uint32_t cols, uint32_t src_rs, uint32_t width, uint32_t R, uint32_t normed, uint32_t rot, uint32_t layout, float eps,
                                float base, uint32_t norm_group, float* qsrc, const WT* __restrict__ qw, uint32_t q_heads, uint32_t temp_every, float temp_coef,
-                               uint32_t hrot, const float* __restrict__ freqs) {
+                               uint32_t hrot, const float* __restrict__ freqs, uint32_t horder, float* __restrict__ pooled, uint32_t pool, uint32_t pool_rows) {
     pdl_enter();
+    if (pooled && blockIdx.x == gridDim.x - 1) {       // single-token steps: one more CTA averages the block that ended just before this token
+        pool_block(pooled, cache, ctl, 1u, cols, width, R, pool, pool_rows, 0u, threadIdx.x, blockDim.x);
+        return;
+    }
     __shared__ float sh[32];
     extern __shared__ float cs_sn[];                   // head rotary: cosine | sine of the token's hrot / 2 angles, shared by all heads
     const uint32_t t = blockIdx.x;
@@ -79,9 +106,10 @@ __global__ void k_cache_append(float* __restrict__ cache, const float* __restric
     float* row = cache + ((size_t)slot * R + pos % R) * width;
     const float* s = src + (size_t)t * src_rs;
     if (hrot) {
-        // Every key head (and query head) is first turned by the token's position on its first hrot values, then divided by the
-        // root mean square of the TURNED vector and weighted: rotary and norm of a head in one pass over it.  One warp per head;
-        // a lane turns whole pairs, so turning in place (the query heads) has no hazard between lanes.
+        // Rotary and norm of every key head (and query head) in one pass over it: horder 0 turns the head by the token's position on
+        // its first hrot values, then divides by the root mean square of the TURNED vector and weights it; 1 norms and weights the
+        // head first, then turns it; 2 only turns it.  One warp per head; a lane turns whole pairs, so turning in place (the query
+        // heads) has no hazard between lanes.
         const uint32_t hh = hrot / 2;
         for (uint32_t i = threadIdx.x; i < hh; i += blockDim.x) {
             float sn, cs;
@@ -97,14 +125,24 @@ __global__ void k_cache_append(float* __restrict__ cache, const float* __restric
             const float* v = key ? s + (size_t)hd * norm_group : qsrc + (size_t)t * src_rs + (size_t)(hd - n_key) * norm_group;
             float* d = key ? row + (size_t)hd * norm_group : qsrc + (size_t)t * src_rs + (size_t)(hd - n_key) * norm_group;
             const WT* w = key ? nw_ : qw;
-            float q = 0.0f;
+            float q = 0.0f, pre = 1.0f;
+            if (horder == 1) {
+                for (uint32_t c = lane; c < norm_group; c += 32) q = fmaf(v[c], v[c], q);
+                pre = (key ? 1.0f : temp) / sqrtf(warp_sum(q) / (float)norm_group + eps);
+            }
             for (uint32_t i = lane; i < hh; i += 32) {
                 const uint32_t a = layout == 0 ? 2 * i : i, b = layout == 0 ? 2 * i + 1 : i + hh;
-                const float u = v[a], x = v[b], ru = u * cs_sn[i] - x * cs_sn[hh + i], rx = x * cs_sn[i] + u * cs_sn[hh + i];
+                float u = v[a], x = v[b];
+                if (horder == 1) { u *= pre * wld(w, a); x *= pre * wld(w, b); }
+                const float ru = u * cs_sn[i] - x * cs_sn[hh + i], rx = x * cs_sn[i] + u * cs_sn[hh + i];
                 d[a] = ru; d[b] = rx;
                 q = fmaf(ru, ru, fmaf(rx, rx, q));
             }
-            for (uint32_t c = hrot + lane; c < norm_group; c += 32) { const float x = v[c]; d[c] = x; q = fmaf(x, x, q); }
+            for (uint32_t c = hrot + lane; c < norm_group; c += 32) {
+                const float x = horder == 1 ? v[c] * pre * wld(w, c) : v[c];
+                d[c] = x; q = fmaf(x, x, q);
+            }
+            if (horder) continue;
             const float mult = (key ? 1.0f : temp) / sqrtf(warp_sum(q) / (float)norm_group + eps);
             __syncwarp();
             for (uint32_t c = lane; c < norm_group; c += 32) d[c] = d[c] * mult * wld(w, c);
@@ -153,10 +191,12 @@ __global__ void k_cache_append(float* __restrict__ cache, const float* __restric
 // ── CACHED_ATTENTION ─────────────────────────────────────────────────────────────────────────────────────────────
 // first position a query at p can see
 __device__ __forceinline__ uint32_t mask_low(uint32_t p, uint32_t kind, uint32_t size) {
-    if (kind == 1) return p + 1 >= size ? p + 1 - size : 0;
+    if (kind == 1 || kind == 3) return p + 1 >= size ? p + 1 - size : 0;
     if (kind == 2) return p - p % size;
     return 0;
 }
+// mask 3: beside its window a query at p sees the mean row of every block of `pool` positions that lies wholly before the window
+__device__ __forceinline__ uint32_t pooled_seen(uint32_t p, uint32_t size, uint32_t pool) { return p + 1 > size ? (p + 1 - size) / pool : 0; }
 struct CaArgs {
     float* dst; const float* q; const float* kc; const float* vc; const float* ctl;
     uint32_t T, H, G, maps, dk, dv, q_rs, q_off, kw, k_off, vw, v_off, R, kind, size;
@@ -168,6 +208,8 @@ struct CaArgs {
     uint32_t sink_bf16;    // its weight type
     float out_scale;       // the result is multiplied by it
     uint32_t dst_rs;       // row stride of dst (its first column is folded into the pointer)
+    const float* kp; const float* vp;   // POOL: pooled rows [slots, pool_rows, kw] (laid out like the cache's), their key and value columns
+    uint32_t pool, pool_rows;
     uint32_t unslotted;    // the caches belong to the step (rows recomputed by the program), not to a state slot
 };
 __device__ __forceinline__ uint32_t ca_slot(const CaArgs& a) { return a.unslotted ? 0u : (uint32_t)ctl_word(a.ctl, ZG_CTL_SLOT); }
@@ -186,7 +228,32 @@ __device__ __forceinline__ float ca_inv_sum(const CaArgs& a, uint32_t hm, float 
 // weight of a visible key under the unnormalised kind
 __device__ __forceinline__ float ca_sigmoid(float s) { return __frcp_rn(1.0f + expf(-s)); }
 constexpr int kCaMaxDv = 1024;   // 32 channels per lane in the per-query kernel
+// Keys as a kernel counts them: positions of the cache, or (POOL) the pooled blocks some row of the tile can see, followed by the
+// positions from k_lo on.  One softmax runs over both.
+template <bool POOL>
+struct CaKeys {
+    const float* cache; const float* pooled;
+    uint32_t R, width, k_lo, n_pool;
+    __device__ __forceinline__ uint32_t first() const { return POOL ? 0u : k_lo; }
+    __device__ __forceinline__ uint32_t count(uint32_t p_max) const { return p_max - k_lo + 1 + (POOL ? n_pool : 0u); }
+    __device__ __forceinline__ bool is_pooled(uint32_t u) const { return POOL && u < n_pool; }
+    __device__ __forceinline__ uint32_t position(uint32_t u) const { return POOL ? u - n_pool + k_lo : u; }
+    __device__ __forceinline__ const float* row(uint32_t u) const { return is_pooled(u) ? pooled + (size_t)u * width : cache + (size_t)(position(u) % R) * width; }
+    // whether a row at position p, whose window starts at lo and that sees nb blocks, sees key u
+    __device__ __forceinline__ bool seen(uint32_t u, uint32_t p, uint32_t lo, uint32_t nb) const {
+        if (is_pooled(u)) return u < nb;
+        const uint32_t j = position(u);
+        return j <= p && j >= lo;
+    }
+};
+template <bool POOL>
+__device__ __forceinline__ CaKeys<POOL> ca_keys(const float* cache, const float* pooled, uint32_t R, uint32_t width, uint32_t k_lo, uint32_t n_pool) {
+    CaKeys<POOL> k;
+    k.cache = cache; k.pooled = pooled; k.R = R; k.width = width; k.k_lo = k_lo; k.n_pool = POOL ? n_pool : 0u;
+    return k;
+}
 // Any shape: one warp per (token, head, map); 32 keys at a time, lane = key for the scores, lane = channel for the sum.
+template <bool POOL>
 __global__ void k_cached_attention(CaArgs a) {
     pdl_enter();
     extern __shared__ float sq[];                      // [warps][dk]
@@ -203,35 +270,40 @@ __global__ void k_cached_attention(CaArgs a) {
     __syncwarp();
     const float* kbase = a.kc + (size_t)slot * a.R * a.kw + a.k_off + (size_t)(g * a.maps + m) * a.dk;
     const float* vbase = a.vc + (size_t)slot * a.R * a.vw + a.v_off + (size_t)g * a.dv;
+    const uint32_t n_pool = POOL ? min(pooled_seen(p, a.size, a.pool), a.pool_rows) : 0u;
+    const size_t pool_slot = POOL ? (size_t)slot * a.pool_rows * a.kw : 0;
+    const CaKeys<POOL> keys = ca_keys<POOL>(kbase, POOL ? a.kp + pool_slot + (size_t)(g * a.maps + m) * a.dk : nullptr, a.R, a.kw, lo, n_pool);
+    const CaKeys<POOL> vals = ca_keys<POOL>(vbase, POOL ? a.vp + pool_slot + (size_t)g * a.dv : nullptr, a.R, a.vw, lo, n_pool);
+    const uint32_t u_begin = keys.first(), u_end = u_begin + keys.count(p);
     float mx = -INFINITY, l = 0.0f;
     float acc[kCaMaxDv / 32];
 #pragma unroll
     for (int i = 0; i < kCaMaxDv / 32; i++) acc[i] = 0.0f;
-    for (uint32_t j0 = lo; j0 <= p; j0 += 32) {
-        const uint32_t j = j0 + lane;
+    for (uint32_t u0 = u_begin; u0 < u_end; u0 += 32) {
+        const uint32_t u = u0 + lane;
         float s = -INFINITY;
-        if (j <= p) {
-            const float* k = kbase + (size_t)(j % a.R) * a.kw;
+        if (u < u_end) {
+            const float* k = keys.row(u);
             float d = 0.0f;
             for (uint32_t c = 0; c < a.dk; c++) d = fmaf(q[c], k[c], d);
             s = ca_score(a, d);
-            if (a.tab) s += a.tab[(size_t)hm * a.tab_rs + (p - j)];
+            if (!POOL && a.tab) s += a.tab[(size_t)hm * a.tab_rs + (p - u)];
         }
         float corr = 1.0f, e;
-        if (a.wkind) e = j <= p ? ca_sigmoid(s) : 0.0f;
+        if (a.wkind) e = u < u_end ? ca_sigmoid(s) : 0.0f;
         else {
-            const float m_new = fmaxf(mx, warp_max(s));    // finite: key j0 is visible
+            const float m_new = fmaxf(mx, warp_max(s));    // finite: key u0 is visible
             corr = expf(mx - m_new);
-            e = j <= p ? expf(s - m_new) : 0.0f;
+            e = u < u_end ? expf(s - m_new) : 0.0f;
             l = l * corr + warp_sum(e);
             mx = m_new;
         }
-        const uint32_t cnt = min(32u, p - j0 + 1);
+        const uint32_t cnt = min(32u, u_end - u0);
 #pragma unroll
         for (int i = 0; i < kCaMaxDv / 32; i++) acc[i] *= corr;
         for (uint32_t jj = 0; jj < cnt; jj++) {
             const float pj = __shfl_sync(0xffffffffu, e, jj);
-            const float* v = vbase + (size_t)((j0 + jj) % a.R) * a.vw;
+            const float* v = vals.row(u0 + jj);
 #pragma unroll
             for (int i = 0; i < kCaMaxDv / 32; i++) {
                 const uint32_t c = lane + 32 * i;
@@ -266,7 +338,7 @@ __device__ __forceinline__ void copy16(float* dst, const float* src, bool on) {
     const int n = on ? 16 : 0;
     asm volatile("cp.async.cg.shared.global [%0], [%1], 16, %2;" ::"r"(d), "l"(src), "r"(n) : "memory");
 }
-template <int OC>
+template <int OC, bool POOL>
 __global__ void __launch_bounds__(kCtThreads) k_cached_attention_tiled(CaArgs a, uint32_t rh, uint32_t n_tiles, uint32_t splits, float* __restrict__ part) {
     pdl_enter();
     constexpr int DV = 16 * OC, KP = kCtDS + 4, PP = kCtBK + 4;
@@ -287,12 +359,16 @@ __global__ void __launch_bounds__(kCtThreads) k_cached_attention_tiled(CaArgs a,
     const uint32_t total = a.T * rh, r0 = tile * kCtBQ, nq = min((uint32_t)kCtBQ, total - r0);
     const uint32_t p_min = pos0 + r0 / rh, p_max = pos0 + (r0 + nq - 1) / rh;
     const uint32_t k_lo = mask_low(p_min, a.kind, a.size);
-    const uint32_t n_keys = p_max - k_lo + 1, per = (n_keys + splits - 1) / splits;
-    const uint32_t k_begin = k_lo + blockIdx.z * per, k_end = min(p_max + 1, k_begin + per);   // this CTA's keys [k_begin, k_end)
     const float* kbase = a.kc + (size_t)slot * a.R * a.kw + a.k_off + (size_t)gm * a.dk;
     const float* vbase = a.vc + (size_t)slot * a.R * a.vw + a.v_off + (size_t)g * a.dv + (size_t)vs * DV;
+    const uint32_t n_pool = POOL ? min(pooled_seen(p_max, a.size, a.pool), a.pool_rows) : 0u;
+    const size_t pool_slot = POOL ? (size_t)slot * a.pool_rows * a.kw : 0;
+    const CaKeys<POOL> keys = ca_keys<POOL>(kbase, POOL ? a.kp + pool_slot + (size_t)gm * a.dk : nullptr, a.R, a.kw, k_lo, n_pool);
+    const CaKeys<POOL> vals = ca_keys<POOL>(vbase, POOL ? a.vp + pool_slot + (size_t)g * a.dv + (size_t)vs * DV : nullptr, a.R, a.vw, k_lo, n_pool);
+    const uint32_t n_keys = keys.count(p_max), per = (n_keys + splits - 1) / splits;
+    const uint32_t k_begin = keys.first() + blockIdx.z * per, k_end = min(keys.first() + n_keys, k_begin + per);   // this CTA's keys [k_begin, k_end)
     const uint32_t v_cols = min((uint32_t)DV, a.dv - vs * DV);
-    uint32_t p_r[4], lo_r[4];
+    uint32_t p_r[4], lo_r[4], nb_r[4];
     bool ok_r[4];
     const float* tab_r[4];                             // the row's line of the score table, so that tab_r[p - j] is the entry of key j
 #pragma unroll
@@ -301,6 +377,7 @@ __global__ void __launch_bounds__(kCtThreads) k_cached_attention_tiled(CaArgs a,
         ok_r[i] = r < total;
         p_r[i] = pos0 + (ok_r[i] ? r / rh : 0);
         lo_r[i] = mask_low(p_r[i], a.kind, a.size);
+        nb_r[i] = POOL ? pooled_seen(p_r[i], a.size, a.pool) : 0u;
         tab_r[i] = a.tab ? a.tab + (size_t)((g * rh + (ok_r[i] ? r % rh : 0)) * a.maps + m) * a.tab_rs : nullptr;
     }
     auto load_q = [&](uint32_t d0, uint32_t stage) {
@@ -315,14 +392,14 @@ __global__ void __launch_bounds__(kCtThreads) k_cached_attention_tiled(CaArgs a,
         for (uint32_t i = tid; i < kCtBK * (kCtDS / 4); i += kCtThreads) {
             const uint32_t rr = i / (kCtDS / 4), c4 = i % (kCtDS / 4);
             const bool on = s0 + rr < k_end && d0 + 4 * c4 < a.dk;
-            copy16(Ks + stage * kCtBK * KP + rr * KP + 4 * c4, on ? kbase + (size_t)((s0 + rr) % a.R) * a.kw + d0 + 4 * c4 : kbase, on);
+            copy16(Ks + stage * kCtBK * KP + rr * KP + 4 * c4, on ? keys.row(s0 + rr) + d0 + 4 * c4 : kbase, on);
         }
     };
     auto load_v = [&](uint32_t s0) {
         for (uint32_t i = tid; i < kCtBK * (DV / 4); i += kCtThreads) {
             const uint32_t rr = i / (DV / 4), c4 = i % (DV / 4);
             const bool on = s0 + rr < k_end && 4 * c4 < v_cols;
-            copy16(Vs + rr * DV + 4 * c4, on ? vbase + (size_t)((s0 + rr) % a.R) * a.vw + 4 * c4 : vbase, on);
+            copy16(Vs + rr * DV + 4 * c4, on ? vals.row(s0 + rr) + 4 * c4 : vbase, on);
         }
     };
     float o[4][OC], m_run[4], l_run[4];
@@ -388,9 +465,9 @@ __global__ void __launch_bounds__(kCtThreads) k_cached_attention_tiled(CaArgs a,
 #pragma unroll
             for (int c = 0; c < 4; c++) {
                 const uint32_t j = s0 + tx + 16 * c;
-                const bool seen = ok_r[r] && j <= p_r[r] && j >= lo_r[r] && j < k_end;
+                const bool seen = ok_r[r] && j < k_end && keys.seen(j, p_r[r], lo_r[r], nb_r[r]);
                 float sv = seen ? ca_score(a, sc[r][c]) : -INFINITY;
-                if (seen && tab_r[r]) sv += tab_r[r][p_r[r] - j];
+                if (!POOL && seen && tab_r[r]) sv += tab_r[r][p_r[r] - j];
                 sc[r][c] = sv;
                 rmax = fmaxf(rmax, sv);
             }
@@ -487,7 +564,7 @@ __global__ void __launch_bounds__(128) k_cached_attention_merge(CaArgs a, const 
 // shuffles; for the weighted sum thread t owns value columns t + 256 i of all rows.  Where the value row is the head of the
 // key row itself (a latent that serves as both), it is not loaded twice.
 constexpr int kCfRows = 16, kCfKeys = 32, kCfThreads = 256, kCfParts = kCfThreads / 32;
-template <int CI>
+template <int CI, bool POOL>
 __global__ void __launch_bounds__(kCfThreads) k_cached_attention_few(CaArgs a, uint32_t rh, uint32_t splits, float* __restrict__ part, uint32_t alias) {
     pdl_enter();
     extern __shared__ __align__(16) float sm[];
@@ -504,12 +581,16 @@ __global__ void __launch_bounds__(kCfThreads) k_cached_attention_few(CaArgs a, u
     const uint32_t pos0 = (uint32_t)ctl_word(a.ctl, ZG_CTL_POS), slot = ca_slot(a);
     const uint32_t total = a.T * rh, p_max = pos0 + a.T - 1;
     const uint32_t k_lo = mask_low(pos0, a.kind, a.size);
-    const uint32_t n_keys = p_max - k_lo + 1, per = (n_keys + splits - 1) / splits;
-    const uint32_t k_begin = k_lo + blockIdx.y * per, k_end = min(p_max + 1, k_begin + per);
     const float* kbase = a.kc + (size_t)slot * a.R * a.kw + a.k_off + (size_t)gm * a.dk;
     const float* vbase = a.vc + (size_t)slot * a.R * a.vw + a.v_off + (size_t)g * a.dv;
+    const uint32_t n_pool = POOL ? min(pooled_seen(p_max, a.size, a.pool), a.pool_rows) : 0u;
+    const size_t pool_slot = POOL ? (size_t)slot * a.pool_rows * a.kw : 0;
+    const CaKeys<POOL> keys = ca_keys<POOL>(kbase, POOL ? a.kp + pool_slot + (size_t)gm * a.dk : nullptr, a.R, a.kw, k_lo, n_pool);
+    const CaKeys<POOL> vals = ca_keys<POOL>(vbase, POOL ? a.vp + pool_slot + (size_t)g * a.dv : nullptr, a.R, a.vw, k_lo, n_pool);
+    const uint32_t n_keys = keys.count(p_max), per = (n_keys + splits - 1) / splits;
+    const uint32_t k_begin = keys.first() + blockIdx.y * per, k_end = min(keys.first() + n_keys, k_begin + per);
     const bool ok = row < total;
-    const uint32_t p_r = pos0 + (ok ? row / rh : 0), lo_r = mask_low(p_r, a.kind, a.size);
+    const uint32_t p_r = pos0 + (ok ? row / rh : 0), lo_r = mask_low(p_r, a.kind, a.size), nb_r = POOL ? pooled_seen(p_r, a.size, a.pool) : 0u;
     const float* tab_r = a.tab ? a.tab + (size_t)((g * rh + (ok ? row % rh : 0)) * a.maps + m) * a.tab_rs : nullptr;
     const uint32_t dk4 = a.dk / 4, dv4 = a.dv / 4;
     const uint32_t chunk4 = (dk4 + kCfParts - 1) / kCfParts, d_begin = 4 * min(dk4, warp * chunk4), d_end = 4 * min(dk4, (warp + 1) * chunk4);
@@ -528,12 +609,12 @@ __global__ void __launch_bounds__(kCfThreads) k_cached_attention_few(CaArgs a, u
         __syncthreads();                               // the previous keys' readers are done
         for (uint32_t i = tid; i < kCfKeys * dk4; i += kCfThreads) {
             const uint32_t kk = i / dk4, c4 = i % dk4;
-            copy16(Ks + kk * KP + 4 * c4, kk < nk ? kbase + (size_t)((s0 + kk) % a.R) * a.kw + 4 * c4 : kbase, kk < nk);
+            copy16(Ks + kk * KP + 4 * c4, kk < nk ? keys.row(s0 + kk) + 4 * c4 : kbase, kk < nk);
         }
         if (!alias)
             for (uint32_t i = tid; i < nk * dv4; i += kCfThreads) {
                 const uint32_t kk = i / dv4, c4 = i % dv4;
-                copy16(Vs + kk * VP + 4 * c4, vbase + (size_t)((s0 + kk) % a.R) * a.vw + 4 * c4, true);
+                copy16(Vs + kk * VP + 4 * c4, vals.row(s0 + kk) + 4 * c4, true);
             }
         asm volatile("cp.async.commit_group;" ::: "memory");   // every load of the share is in flight at once: one round trip
         asm volatile("cp.async.wait_group 0;" ::: "memory");
@@ -571,9 +652,9 @@ __global__ void __launch_bounds__(kCfThreads) k_cached_attention_few(CaArgs a, u
             float d = 0.0f;
 #pragma unroll
             for (int w = 0; w < kCfParts; w++) d += Sp[(w * kCfRows + row) * kCfKeys + kk];
-            const bool seen = ok && kk < nk && j <= p_r && j >= lo_r;
+            const bool seen = ok && kk < nk && keys.seen(j, p_r, lo_r, nb_r);
             sv[u] = seen ? ca_score(a, d) : -INFINITY;
-            if (seen && tab_r) sv[u] += tab_r[p_r - j];
+            if (!POOL && seen && tab_r) sv[u] += tab_r[p_r - j];
         }
         float rmax = fmaxf(sv[0], sv[1]);
 #pragma unroll
@@ -645,10 +726,11 @@ template <int OC>
 static void launch_cached_attention_tiled(const CaArgs& a, uint32_t splits, float* part, cudaStream_t st) {
     constexpr int DV = 16 * OC;
     const size_t smem = ((size_t)(a.dk <= (uint32_t)kCtDS ? 1 : 2) * kCtBQ * kCtDS + (size_t)2 * kCtBK * (kCtDS + 4) + (size_t)kCtBQ * (kCtBK + 4) + (size_t)kCtBK * DV) * sizeof(float);
-    static size_t most = 0;
-    if (smem > most) { cudaFuncSetAttribute(k_cached_attention_tiled<OC>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem); most = smem; }
+    auto kernel = a.pool ? k_cached_attention_tiled<OC, true> : k_cached_attention_tiled<OC, false>;
+    static size_t most[2] = {0, 0};
+    if (smem > most[a.pool != 0]) { cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem); most[a.pool != 0] = smem; }
     const uint32_t rh = a.H / a.G, n_tiles = (a.T * rh + kCtBQ - 1) / kCtBQ, n_vs = (a.dv + DV - 1) / DV;
-    launch_pdl(k_cached_attention_tiled<OC>, dim3(n_tiles, a.G * a.maps * n_vs, splits), dim3(kCtThreads), smem, st, a, rh, n_tiles, splits, part);
+    launch_pdl(kernel, dim3(n_tiles, a.G * a.maps * n_vs, splits), dim3(kCtThreads), smem, st, a, rh, n_tiles, splits, part);
 }
 static bool ca_aligned(const ZgSeqOp& s) {
     return s.n[4] % 4 == 0 && s.n[5] % 4 == 0 && s.n[6] % 4 == 0 && s.n[7] % 4 == 0 && s.n[8] % 4 == 0 && s.off[0] % 4 == 0 && s.off[1] % 4 == 0 && s.off[2] % 4 == 0;
@@ -656,17 +738,22 @@ static bool ca_aligned(const ZgSeqOp& s) {
 static bool ca_few(const ZgSeqOp& s) {
     return ca_aligned(s) && s.n[0] * (s.n[1] / s.n[2]) <= (uint32_t)kCfRows && cf_smem(s.n[4], s.n[5], cf_alias(s)) <= 200 * 1024;
 }
+// keys a step's rows can see at most
+static uint32_t ca_reach(const ZgSeqOp& s) {
+    const uint32_t tokens = s.off[3] ? min(s.n[9], s.off[4] + s.n[0]) : s.n[9];
+    return s.off[3] == 3 ? tokens + s.off[6] : tokens;
+}
 // key shares per row tile: few CTAs and a long cache (decoding) spread over more of them
 static uint32_t ca_splits(const ZgSeqOp& s) {
     if (!ca_aligned(s)) return 1;
     if (ca_few(s)) {
-        const uint32_t reach = s.off[3] ? min(s.n[9], s.off[4] + s.n[0]) : s.n[9];
+        const uint32_t reach = ca_reach(s);
         const uint32_t S = (reach + kCfKeys - 1) / kCfKeys;
         return S < 2 ? 1 : (S > (uint32_t)kCtMaxSplits ? (uint32_t)kCtMaxSplits : S);
     }
     const uint32_t rh = s.n[1] / s.n[2], n_tiles = (s.n[0] * rh + kCtBQ - 1) / kCtBQ, dvs = s.n[5] > 256 ? 512 : (s.n[5] > 128 ? 256 : 128);
     const uint32_t ctas = n_tiles * s.n[2] * s.n[3] * ((s.n[5] + dvs - 1) / dvs);
-    const uint32_t reach = s.off[3] ? min(s.n[9], s.off[4] + s.n[0]) : s.n[9];     // keys a row can see at most
+    const uint32_t reach = ca_reach(s);
     uint32_t S = 160 / (ctas ? ctas : 1), most = reach / kCtMinShare;
     if (S > most) S = most;
     return S < 2 ? 1 : (S > (uint32_t)kCtMaxSplits ? (uint32_t)kCtMaxSplits : S);
@@ -858,7 +945,9 @@ bool zg_mix_op_valid(const ZgOp& op, const size_t* elems, size_t n_bufs, char* w
             if (!T || !cols || R < T || s.off[0] + cols > srs || s.off[1] + cols > width || normed + rot > cols || rot % 2 || s.n[8] > 1) return fail("cache_append: shape");
             if (!have(0) || elems[s.buf[0]] < R * width || !fits(1, 0, (T - 1) * srs + s.off[0] + cols) || !fits(2, 0, ZG_CTL_IDS)) return fail("cache_append: extent");
             if (normed && s.n[9] && normed % s.n[9]) return fail("cache_append: norm groups");
-            if (normed && !wfits(3, s.n[7], s.off[2], s.n[9] ? s.n[9] : normed)) return fail("cache_append: norm weight");
+            const bool turn_only = s.n[13] == 2;
+            if (s.n[13] > 2 || (s.n[13] && !s.n[10])) return fail("cache_append: order of norm and rotation");
+            if (normed && !turn_only && !wfits(3, s.n[7], s.off[2], s.n[9] ? s.n[9] : normed)) return fail("cache_append: norm weight");
             if (rot && !(s.f[1] > 0.0f)) return fail("cache_append: rotary base");
             if (s.n[10]) {     // rotary inside every normed head, before its norm
                 if (!normed || !s.n[9] || rot || s.n[10] % 2 || s.n[10] > s.n[9]) return fail("cache_append: head rotary");
@@ -866,15 +955,19 @@ bool zg_mix_op_valid(const ZgOp& op, const size_t* elems, size_t n_bufs, char* w
             }
             if (s.off[5]) {    // query heads normed in place in the source rows
                 const size_t qh = s.off[5], hd = s.n[9];
-                if (!normed || !hd || s.off[3] + qh * hd > srs || !fits(1, 0, (T - 1) * srs + s.off[3] + qh * hd) || !wfits(3, s.n[7], s.off[4], hd)) return fail("cache_append: query heads");
+                if (!normed || !hd || s.off[3] + qh * hd > srs || !fits(1, 0, (T - 1) * srs + s.off[3] + qh * hd) || (!turn_only && !wfits(3, s.n[7], s.off[4], hd))) return fail("cache_append: query heads");
                 if (s.off[3] < s.off[0] + cols && s.off[0] < s.off[3] + qh * hd) return fail("cache_append: query heads overlap the appended columns");
+            }
+            if (s.n[11]) {     // pooled blocks of the appended rows
+                if (R < T + s.n[11] || !s.n[12] || !have(5) || elems[s.buf[5]] < (size_t)s.n[12] * width || s.buf[5] == s.buf[0] || s.buf[5] == s.buf[1])
+                    return fail("cache_append: pooled blocks");
             }
             return true;
         }
         case ZG_OP_CACHED_ATTENTION: {
             const size_t T = s.n[0], H = s.n[1], G = s.n[2], maps = s.n[3], dk = s.n[4], dv = s.n[5], qrs = s.n[6], kw = s.n[7], vw = s.n[8], R = s.n[9];
             const uint32_t kind = s.off[3], size = s.off[4];
-            if (!T || !H || !G || H % G || !maps || !dk || !dv || dv > kCaMaxDv || kind > 2 || (kind && !size)) return fail("cached_attention: shape");
+            if (!T || !H || !G || H % G || !maps || !dk || !dv || dv > kCaMaxDv || kind > 3 || (kind && !size)) return fail("cached_attention: shape");
             if (R < T) return fail("cached_attention: cache rows");   // the caller sizes R for what the mask reaches and bounds the positions
             if (s.off[0] + H * maps * dk > qrs || s.off[1] + G * maps * dk > kw || s.off[2] + G * dv > vw) return fail("cached_attention: columns");
             const size_t drs = s.n[10] ? s.n[10] : H * maps * dv;
@@ -885,6 +978,10 @@ bool zg_mix_op_valid(const ZgOp& op, const size_t* elems, size_t n_bufs, char* w
                 return fail("cached_attention: extent");
             if (s.buf[0] == s.buf[1]) return fail("cached_attention: in place");
             if (s.off[5] > 1) return fail("cached_attention: weights");
+            if (kind == 3) {                           // pooled rows, laid out like the one cache that holds keys and values
+                if (!s.n[15] || s.off[5] || s.n[14] || s.buf[5] != ZG_NO_BUF || s.buf[2] != s.buf[3] || kw != vw || !have(7) || elems[s.buf[7]] < (size_t)s.off[6] * kw || !s.off[6])
+                    return fail("cached_attention: pooled rows");
+            }
             if (s.buf[5] != ZG_NO_BUF) {               // the table must cover every distance the mask lets a query reach
                 const size_t reach = kind == 0 ? R : (size < R ? size : R);
                 if (s.off[6] < reach || !fits(5, 0, H * maps * (size_t)s.off[6])) return fail("cached_attention: score table");
@@ -926,7 +1023,7 @@ bool zg_mix_op_valid(const ZgOp& op, const size_t* elems, size_t n_bufs, char* w
 }
 
 uint32_t zg_mix_op_writes(uint32_t tag) {
-    if (tag == ZG_OP_CACHE_APPEND) return 1u | (1u << 1);   // the source rows too: query heads may be normed in place
+    if (tag == ZG_OP_CACHE_APPEND) return 1u | (1u << 1) | (1u << 5);   // the source rows too: query heads may be normed in place; pooled blocks, where named
     return tag == ZG_OP_TOKEN_SHIFT ? (1u | (1u << 3)) : 1u;
 }
 
@@ -961,13 +1058,22 @@ bool zg_launch_mix_op(const ZgOp& op, float* const* bufs, float* scratch, cudaSt
             ZG_SEQ_CHECK();
             return true;
         }
-        case ZG_OP_CACHE_APPEND:
-            ZG_SEQ_WDT(s.n[5] ? s.n[7] : ZG_W_F32, launch_pdl(k_cache_append<WT>, dim3(s.n[0]), dim3(s.off[5] ? 256 : 128), (size_t)s.n[10] * sizeof(float), st, bufs[s.buf[0]] + s.off[1], bufs[s.buf[1]] + s.off[0], bufs[s.buf[2]],
-                                                             s.n[5] ? wptr<WT>(bufs, s.buf[3], s.off[2]) : nullptr, s.n[1], s.n[2], s.n[3], s.n[4], s.n[5], s.n[6], s.n[8], s.f[0], s.f[1], s.n[9],
-                                                             s.off[5] ? bufs[s.buf[1]] + s.off[3] : nullptr, s.off[5] ? wptr<WT>(bufs, s.buf[3], s.off[4]) : nullptr, s.off[5], s.off[6], s.f[2],
-                                                             s.n[10], s.n[10] && s.buf[4] != ZG_NO_BUF ? (const float*)(bufs[s.buf[4]] + s.off[7]) : (const float*)nullptr));
+        case ZG_OP_CACHE_APPEND: {
+            float* pooled = s.n[11] ? bufs[s.buf[5]] + s.off[1] : nullptr;
+            const bool turn_only = s.n[13] == 2;
+            ZG_SEQ_WDT(s.n[5] ? s.n[7] : ZG_W_F32, launch_pdl(k_cache_append<WT>, dim3(s.n[0] + (pooled && s.n[0] == 1 ? 1 : 0)), dim3(s.off[5] ? 256 : 128), (size_t)s.n[10] * sizeof(float), st, bufs[s.buf[0]] + s.off[1], bufs[s.buf[1]] + s.off[0], bufs[s.buf[2]],
+                                                             s.n[5] && !turn_only ? wptr<WT>(bufs, s.buf[3], s.off[2]) : nullptr, s.n[1], s.n[2], s.n[3], s.n[4], s.n[5], s.n[6], s.n[8], s.f[0], s.f[1], s.n[9],
+                                                             s.off[5] ? bufs[s.buf[1]] + s.off[3] : nullptr, s.off[5] && !turn_only ? wptr<WT>(bufs, s.buf[3], s.off[4]) : nullptr, s.off[5], s.off[6], s.f[2],
+                                                             s.n[10], s.n[10] && s.buf[4] != ZG_NO_BUF ? (const float*)(bufs[s.buf[4]] + s.off[7]) : (const float*)nullptr, s.n[13],
+                                                             s.n[0] == 1 ? pooled : (float*)nullptr, s.n[11], s.n[12]));
             ZG_SEQ_CHECK();
+            if (pooled && s.n[0] > 1) {
+                launch_pdl(k_block_pool, dim3((s.n[0] - 1) / s.n[11] + 1, (s.n[1] + 127) / 128), dim3(128), 0, st, pooled, (const float*)(bufs[s.buf[0]] + s.off[1]), (const float*)bufs[s.buf[2]],
+                           s.n[0], s.n[1], s.n[3], s.n[4], s.n[11], s.n[12]);
+                ZG_SEQ_CHECK();
+            }
             return true;
+        }
         case ZG_OP_CACHED_ATTENTION: {
             CaArgs a;
             a.dst = bufs[s.buf[0]]; a.q = bufs[s.buf[1]]; a.kc = bufs[s.buf[2]]; a.vc = bufs[s.buf[3]]; a.ctl = bufs[s.buf[4]];
@@ -976,8 +1082,10 @@ bool zg_launch_mix_op(const ZgOp& op, float* const* bufs, float* scratch, cudaSt
             a.tab = s.buf[5] != ZG_NO_BUF ? bufs[s.buf[5]] : nullptr; a.tab_rs = s.off[6]; a.wkind = s.off[5];
             a.cap = s.f[1]; a.out_scale = s.n[13] ? s.f[2] : 1.0f; a.dst_rs = s.n[10] ? s.n[10] : a.H * a.maps * a.dv; a.dst += s.n[11];
             a.sink = nullptr; a.sink_bf16 = s.n[12] == ZG_W_BF16; a.unslotted = s.n[14];
+            a.kp = a.vp = nullptr; a.pool = a.pool_rows = 0;
+            if (a.kind == 3) { a.pool = s.n[15]; a.pool_rows = s.off[6]; a.kp = bufs[s.buf[7]] + a.k_off; a.vp = bufs[s.buf[7]] + a.v_off; }
             if (s.buf[6] != ZG_NO_BUF) a.sink = a.sink_bf16 ? (const void*)wptr<bf16>(bufs, s.buf[6], s.off[7]) : (const void*)wptr<float>(bufs, s.buf[6], s.off[7]);
-            const bool aligned = ca_aligned(s) && ((reinterpret_cast<uintptr_t>(a.q) | reinterpret_cast<uintptr_t>(a.kc) | reinterpret_cast<uintptr_t>(a.vc)) & 15) == 0;
+            const bool aligned = ca_aligned(s) && ((reinterpret_cast<uintptr_t>(a.kp) | reinterpret_cast<uintptr_t>(a.q) | reinterpret_cast<uintptr_t>(a.kc) | reinterpret_cast<uintptr_t>(a.vc)) & 15) == 0;
             if (aligned && ca_few(s)) {
                 const uint32_t S = scratch ? ca_splits(s) : 1, alias = cf_alias(s) ? 1u : 0u;
                 float* part = S > 1 ? scratch : nullptr;
@@ -985,9 +1093,10 @@ bool zg_launch_mix_op(const ZgOp& op, float* const* bufs, float* scratch, cudaSt
                 const dim3 grid(a.G * a.maps, S);
 #define ZG_CF(CI_)                                                                                                                         \
     do {                                                                                                                                   \
-        static size_t most = 48 * 1024;                                                                                                    \
-        if (smem > most) { cudaFuncSetAttribute(k_cached_attention_few<CI_>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem); most = smem; } \
-        launch_pdl(k_cached_attention_few<CI_>, grid, dim3(kCfThreads), smem, st, a, a.H / a.G, S, part, alias);                            \
+        static size_t most[2] = {48 * 1024, 48 * 1024};                                                                                    \
+        auto kernel = a.pool ? k_cached_attention_few<CI_, true> : k_cached_attention_few<CI_, false>;                                     \
+        if (smem > most[a.pool != 0]) { cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem); most[a.pool != 0] = smem; } \
+        launch_pdl(kernel, grid, dim3(kCfThreads), smem, st, a, a.H / a.G, S, part, alias);                            \
     } while (0)
                 if (a.dv <= 256) ZG_CF(1); else if (a.dv <= 512) ZG_CF(2); else ZG_CF(4);
 #undef ZG_CF
@@ -1018,7 +1127,7 @@ bool zg_launch_mix_op(const ZgOp& op, float* const* bufs, float* scratch, cudaSt
                 }
             } else {
                 const uint32_t warps = 4, items = a.T * a.H * a.maps;
-                launch_pdl(k_cached_attention, dim3((items + warps - 1) / warps), dim3(warps * 32), warps * a.dk * sizeof(float), st, a);
+                launch_pdl(a.pool ? k_cached_attention<true> : k_cached_attention<false>, dim3((items + warps - 1) / warps), dim3(warps * 32), warps * a.dk * sizeof(float), st, a);
             }
             ZG_SEQ_CHECK();
             return true;

@@ -43,6 +43,7 @@ __host__ __device__ inline uint32_t ssm_slices(uint32_t N) {
 struct SsmArgs {
     float* dst; const float* xbc; const float* dtl; float* state; const float* ctl;
     uint32_t T, H, G, N, P, x_off, b_off, c_off, dt_off, xbc_rs, dt_rs, vec;
+    uint32_t constant;     // form: the decay is a constant per head (a table dtl[H]), the step size 1, and there is no D x in the read-out
     // Segments of a long step walked side by side (the recurrence is linear in the state).  mode 0: the whole step from the carried
     // state.  mode 1: segment blockIdx.z from an EMPTY state, no read-out; leaves the state it reaches and the product of its decays.
     // mode 2: segment blockIdx.z from the state it really starts from (segment 0: the carried one), with the read-out; the last
@@ -88,7 +89,9 @@ __global__ void __launch_bounds__(kSsmThreads) k_ssm_scan(SsmArgs a, const WT* _
         S[i / 4][(i / 2) % 2][i % 2].y = a.mode == 1 ? 0.0f : from[(2 * i + 1) * kSsmThreads + tid];
     }
     float decay_product = 1.0f;                                          // mode 1, thread 0
-    const float neg_a = -expf(wld(a_log, h)), bias = wld(dt_bias, h), dsk = wld(dskip, h);
+    const bool fixed = a.constant != 0;
+    const float neg_a = fixed ? 0.0f : -expf(wld(a_log, h)), bias = fixed ? 0.0f : wld(dt_bias, h), dsk = fixed ? 0.0f : wld(dskip, h);
+    const float fixed_decay = fixed ? a.dtl[h] : 0.0f;
     const float* bsrc = a.xbc + a.b_off + (size_t)g * a.N;
     const float* csrc = a.xbc + a.c_off + (size_t)g * a.N;
     const float* xsrc = a.xbc + a.x_off + (size_t)h * a.P + (size_t)cb * CPB;
@@ -134,6 +137,7 @@ __global__ void __launch_bounds__(kSsmThreads) k_ssm_scan(SsmArgs a, const WT* _
         fetch_tile(base, 0);
         asm volatile("cp.async.commit_group;" ::: "memory");
         for (uint32_t t = tid; t < span; t += kSsmThreads) {
+            if (fixed) { Dt[t] = 1.0f; Dec[t] = fixed_decay; continue; }
             const float dt = softplusf_(a.dtl[(size_t)(base + t) * a.dt_rs + a.dt_off + h] + bias);
             Dt[t] = dt;
             Dec[t] = expf(neg_a * dt);
@@ -352,9 +356,12 @@ static uint32_t scan_segments(uint32_t T, uint32_t* seg_len) {
 }
 
 // ── GATED_NORM: one CTA per (token, group) ───────────────────────────────────────────────────────────────────────
+// forms (op parameter n7): the gate multiplies what the norm returns instead of what it reads; a sigmoid gate instead of SiLU
+constexpr uint32_t kGateAfter = 1, kGateSigmoid = 2;
+__device__ __forceinline__ float gated_norm_gate(float z, uint32_t form) { return (form & kGateSigmoid) ? sigmoidf_(z) : z * sigmoidf_(z); }
 template <typename WT>
 __global__ void k_gated_norm(float* dst, const float* src, const float* __restrict__ gate, const WT* __restrict__ w, uint32_t cols, uint32_t groups,
-                             uint32_t gate_rs, uint32_t src_rs, uint32_t dst_rs, float eps) {
+                             uint32_t gate_rs, uint32_t src_rs, uint32_t dst_rs, float eps, uint32_t form) {
     pdl_enter();
     __shared__ float sh[32];
     const uint32_t t = blockIdx.x / groups, gi = blockIdx.x % groups, gs = cols / groups, c0 = gi * gs;
@@ -373,7 +380,11 @@ __global__ void k_gated_norm(float* dst, const float* src, const float* __restri
         }
         float q = 0.0f;
 #pragma unroll
-        for (int i = 0; i < kKeep; i++) { v[i] *= z[i] * sigmoidf_(z[i]); q = fmaf(v[i], v[i], q); }
+        for (int i = 0; i < kKeep; i++) {
+            z[i] = gated_norm_gate(z[i], form);
+            if (form & kGateAfter) wv[i] *= z[i]; else v[i] *= z[i];
+            q = fmaf(v[i], v[i], q);
+        }
         const float inv = 1.0f / sqrtf(block_sum(q, sh) / (float)gs + eps);
 #pragma unroll
         for (int i = 0; i < kKeep; i++) {
@@ -384,13 +395,12 @@ __global__ void k_gated_norm(float* dst, const float* src, const float* __restri
     }
     float q = 0.0f;
     for (uint32_t c = threadIdx.x; c < gs; c += blockDim.x) {
-        const float z = gt[c], v = x[c] * (z * sigmoidf_(z));
+        const float v = (form & kGateAfter) ? x[c] : x[c] * gated_norm_gate(gt[c], form);
         q = fmaf(v, v, q);
     }
     const float inv = 1.0f / sqrtf(block_sum(q, sh) / (float)gs + eps);
     for (uint32_t c = threadIdx.x; c < gs; c += blockDim.x) {
-        const float z = gt[c], v = x[c] * (z * sigmoidf_(z));
-        out[c] = v * inv * wld(w, c0 + c);
+        out[c] = x[c] * gated_norm_gate(gt[c], form) * inv * wld(w, c0 + c);
     }
 }
 
@@ -460,9 +470,10 @@ bool zg_rec_op_valid(const ZgOp& op, const size_t* elems, size_t n_bufs, char* w
         case ZG_OP_SSM_SCAN: {
             const size_t T = s.n[0], H = s.n[1], G = s.n[2], N = s.n[3], P = s.n[4], xrs = s.n[5], drs = s.n[6];
             if (!T || !H || !G || H % G || !N || N > (size_t)kSsmMaxN || !P) return fail("ssm_scan: shape");
-            if (s.off[0] + H * P > xrs || s.off[1] + G * N > xrs || s.off[2] + G * N > xrs || s.off[3] + H > drs) return fail("ssm_scan: columns");
-            if (!fits(0, 0, T * H * P) || !fits(1, 0, T * xrs) || !fits(2, 0, T * drs) || !wfits(3, s.n[7], s.off[4], H) || !wfits(3, s.n[7], s.off[5], H) ||
-                !wfits(3, s.n[7], s.off[6], H) || !have(4) || elems[s.buf[4]] < ssm_state_elems((uint32_t)H, (uint32_t)N, (uint32_t)P) || !fits(5, 0, ZG_CTL_IDS))
+            const bool fixed = s.n[8] != 0;        // constant decays: a table instead of the dt rows, no weights
+            if (s.n[8] > 1 || s.off[0] + H * P > xrs || s.off[1] + G * N > xrs || s.off[2] + G * N > xrs || (!fixed && s.off[3] + H > drs)) return fail("ssm_scan: columns");
+            if (!fits(0, 0, T * H * P) || !fits(1, 0, T * xrs) || !fits(2, fixed ? s.off[3] : 0, fixed ? H : T * drs) ||
+                (!fixed && (!wfits(3, s.n[7], s.off[4], H) || !wfits(3, s.n[7], s.off[5], H) || !wfits(3, s.n[7], s.off[6], H))) || !have(4) || elems[s.buf[4]] < ssm_state_elems((uint32_t)H, (uint32_t)N, (uint32_t)P) || !fits(5, 0, ZG_CTL_IDS))
                 return fail("ssm_scan: extent");
             if (s.buf[0] == s.buf[1] || s.buf[0] == s.buf[2]) return fail("ssm_scan: in place");
             return true;
@@ -476,7 +487,7 @@ bool zg_rec_op_valid(const ZgOp& op, const size_t* elems, size_t n_bufs, char* w
         }
         case ZG_OP_GATED_NORM: {
             const size_t T = s.n[0], cols = s.n[1], groups = s.n[2], grs = s.n[3], srs = s.n[5], drs = s.n[6];
-            if (!T || !cols || !groups || cols % groups || srs < cols || drs < cols || s.off[0] + cols > grs) return fail("gated_norm: shape");
+            if (!T || !cols || !groups || cols % groups || srs < cols || drs < cols || s.off[0] + cols > grs || s.n[7] > 3) return fail("gated_norm: shape");
             if (!fits(0, 0, (T - 1) * drs + cols) || !fits(1, 0, (T - 1) * srs + cols) || !fits(2, 0, (T - 1) * grs + s.off[0] + cols) || !wfits(3, s.n[4], s.off[1], cols))
                 return fail("gated_norm: extent");
             return true;
@@ -489,7 +500,7 @@ bool zg_rec_op_valid(const ZgOp& op, const size_t* elems, size_t n_bufs, char* w
         }
         case ZG_OP_RG_LRU: {
             const size_t T = s.n[0], W = s.n[1], urs = s.n[2], grs = s.n[3], bw = s.n[4], bs = s.n[5], yrs = s.n[6], drs = s.n[7];
-            if (!T || !W || !bw || W % bw || bs < bw || drs < W || s.n[9] > 5 || !(s.f[0] > 0.0f)) return fail("rg_lru: shape");
+            if (!T || !W || !bw || W % bw || bs < bw || drs < W || s.n[9] > 6 || !(s.f[0] > 0.0f)) return fail("rg_lru: shape");
             const size_t gspan = (W / bw - 1) * bs + bw;
             if (s.off[0] + W > urs || s.off[1] + gspan > grs || s.off[2] + gspan > grs || s.off[3] + W > yrs) return fail("rg_lru: columns");
             if (!fits(0, 0, (T - 1) * drs + W) || !fits(1, 0, (T - 1) * urs + s.off[0] + W) || !fits(2, 0, (T - 1) * grs + (s.off[1] > s.off[2] ? s.off[1] : s.off[2]) + gspan) ||
@@ -500,7 +511,7 @@ bool zg_rec_op_valid(const ZgOp& op, const size_t* elems, size_t n_bufs, char* w
             return true;
         }
         case ZG_OP_ACTIVATION: {
-            if (!s.n[0] || s.n[1] > 4 || (s.n[1] == 4 && !(s.f[0] > 0.0f))) return fail("activation: shape");
+            if (!s.n[0] || s.n[1] > 5 || (s.n[1] == 4 && !(s.f[0] > 0.0f))) return fail("activation: shape");
             if (!fits(0, 0, s.n[0]) || !fits(1, 0, s.n[0])) return fail("activation: extent");
             return true;
         }
@@ -524,7 +535,8 @@ bool zg_launch_rec_op(const ZgOp& op, float* const* bufs, float* scratch, cudaSt
             SsmArgs a;
             a.dst = bufs[s.buf[0]]; a.xbc = bufs[s.buf[1]]; a.dtl = bufs[s.buf[2]]; a.state = bufs[s.buf[4]]; a.ctl = bufs[s.buf[5]];
             a.T = s.n[0]; a.H = s.n[1]; a.G = s.n[2]; a.N = s.n[3]; a.P = s.n[4]; a.x_off = s.off[0]; a.b_off = s.off[1]; a.c_off = s.off[2]; a.dt_off = s.off[3];
-            a.xbc_rs = s.n[5]; a.dt_rs = s.n[6];
+            a.xbc_rs = s.n[5]; a.dt_rs = s.n[6]; a.constant = s.n[8];
+            if (a.constant) a.dtl += s.off[3];
             const uint32_t NS = ssm_slices(a.N), RQ = ssm_rq(a.N), CPB = kSsmThreads / NS * 2;
             // 16-byte copies when every row of B, C and the CTA's x columns starts on a 16-byte boundary
             a.vec = (a.N % 4 == 0 && a.P % 4 == 0 && a.xbc_rs % 4 == 0 && a.x_off % 4 == 0 && a.b_off % 4 == 0 && a.c_off % 4 == 0 &&
@@ -539,8 +551,8 @@ bool zg_launch_rec_op(const ZgOp& op, float* const* bufs, float* scratch, cudaSt
 #define ZG_SSM(NS_, RQ_)                                                                                                                  \
     ZG_SEQ_WDT(s.n[7], {                                                                                                                  \
         if (smem > 48 * 1024) cudaFuncSetAttribute(k_ssm_scan<WT, NS_, RQ_>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);     \
-        launch_pdl_if(a.T < (uint32_t)kLongWalk, k_ssm_scan<WT, NS_, RQ_>, grid, dim3(kSsmThreads), smem, st, a, wptr<WT>(bufs, s.buf[3], s.off[4]), \
-                      wptr<WT>(bufs, s.buf[3], s.off[5]), wptr<WT>(bufs, s.buf[3], s.off[6]));                                            \
+        launch_pdl_if(a.T < (uint32_t)kLongWalk, k_ssm_scan<WT, NS_, RQ_>, grid, dim3(kSsmThreads), smem, st, a, a.constant ? (const WT*)nullptr : (const WT*)wptr<WT>(bufs, s.buf[3], s.off[4]), \
+                      a.constant ? (const WT*)nullptr : (const WT*)wptr<WT>(bufs, s.buf[3], s.off[5]), a.constant ? (const WT*)nullptr : (const WT*)wptr<WT>(bufs, s.buf[3], s.off[6]));                                            \
     })
 #define ZG_SSM_ANY()                                                                                                                      \
     do {                                                                                                                                  \
@@ -602,7 +614,7 @@ bool zg_launch_rec_op(const ZgOp& op, float* const* bufs, float* scratch, cudaSt
             const uint32_t gs = s.n[1] / s.n[2];
             const uint32_t threads = gs <= 64 ? 32 : (gs <= 512 ? 128 : (gs <= 2048 ? 256 : 512));
             ZG_SEQ_WDT(s.n[4], launch_pdl(k_gated_norm<WT>, dim3(s.n[0] * s.n[2]), dim3(threads), 0, st, bufs[s.buf[0]], bufs[s.buf[1]], bufs[s.buf[2]] + s.off[0],
-                                          wptr<WT>(bufs, s.buf[3], s.off[1]), s.n[1], s.n[2], s.n[3], s.n[5], s.n[6], s.f[0]));
+                                          wptr<WT>(bufs, s.buf[3], s.off[1]), s.n[1], s.n[2], s.n[3], s.n[5], s.n[6], s.f[0], s.n[7]));
             ZG_SEQ_CHECK();
             return true;
         }

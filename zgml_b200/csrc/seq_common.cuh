@@ -61,18 +61,22 @@ __device__ __forceinline__ float sigmoidf_(float z) { return 1.0f / (1.0f + expf
 __device__ __forceinline__ float softplusf_(float z) { return z > 20.0f ? z : log1pf(expf(z)); }
 __device__ __forceinline__ int ctl_word(const float* ctl, int i) { return reinterpret_cast<const int*>(ctl)[i]; }
 // the activations of ACTIVATION and of LINEAR's epilogue: 0 relu(z)^2, 1 silu, 2 gelu (tanh form), 3 relu, 4 smooth cap
-// p * tanh(z / p) (p: the op's activation parameter)
+// p * tanh(z / p) (p: the op's activation parameter), 5 gelu (exact, erf form)
 __device__ __forceinline__ float seq_activation(float z, uint32_t kind, float p = 0.0f) {
     switch (kind) {
         case 0: { const float r = fmaxf(z, 0.0f); return r * r; }
         case 1: return z * sigmoidf_(z);
         case 2: return 0.5f * z * (1.0f + tanhf(0.7978845608028654f * fmaf(0.044715f * z * z, z, z)));
         case 4: return p * tanhf(z / p);
+        case 5: return 0.5f * z * (1.0f + erff(z * 0.7071067811865476f));
         default: return fmaxf(z, 0.0f);
     }
 }
 // epilogue form: act = 0 none, kind + 1 otherwise
 __device__ __forceinline__ float seq_epilogue(float z, uint32_t act, float p = 0.0f) { return act ? seq_activation(z, act - 1, p) : z; }
+// activation of a product's epilogue, applied to the columns [lo, hi) only (a stacked projection whose parts differ)
+struct SeqAct { uint32_t kind; float p; uint32_t lo, hi; };
+__device__ __forceinline__ float seq_epilogue(float z, const SeqAct& a, uint32_t n) { return (a.kind && n >= a.lo && n < a.hi) ? seq_activation(z, a.kind - 1, a.p) : z; }
 
 // 16-byte weight loads (8 bf16 / 4 f32 per lane and trip) when the row start and K allow it
 template <typename WT> struct WVec;

@@ -15,10 +15,19 @@ namespace {
 // ── EMBED ─────────────────────────────────────────────────────────────────────────────────────────────────────────
 template <typename WT>
 __global__ void k_embed(float* __restrict__ dst, const float* __restrict__ ctl, const WT* __restrict__ table, uint32_t D, float scale,
-                        const WT* __restrict__ positions) {
+                        const WT* __restrict__ positions, const WT* __restrict__ bigram, uint32_t buckets, uint32_t mul_prev, uint32_t mul_cur) {
     pdl_enter();
     const uint32_t t = blockIdx.x;
     const size_t row = (size_t)ctl_word(ctl, ZG_CTL_IDS + t) * D;
+    if (bigram) {          // a row chosen by a hash of the previous and the current token, not scaled; a sequence's first token takes the last row
+        const int prev = t ? ctl_word(ctl, ZG_CTL_IDS + t - 1) : ctl_word(ctl, ZG_CTL_PREV);
+        const unsigned long long cur = (unsigned long long)ctl_word(ctl, ZG_CTL_IDS + t);
+        const unsigned long long b = prev < 0 ? (unsigned long long)buckets : ((unsigned long long)prev * mul_prev + cur * mul_cur) % buckets;
+        const size_t brow = (size_t)b * D;
+#pragma unroll 4
+        for (uint32_t c = threadIdx.x; c < D; c += blockDim.x) dst[(size_t)t * D + c] = fmaf(wld(table, row + c), scale, wld(bigram, brow + c));
+        return;
+    }
     if (positions) {       // a learned position row, not scaled
         const size_t prow = ((size_t)ctl_word(ctl, ZG_CTL_POS) + t) * D;
 #pragma unroll 4
@@ -32,7 +41,7 @@ __global__ void k_embed(float* __restrict__ dst, const float* __restrict__ ctl, 
 constexpr int kGemvRows = 8;
 template <typename WT>
 __global__ void k_linear_rows(float* __restrict__ dst, const float* __restrict__ src, const WT* __restrict__ W, const WT* __restrict__ bias,
-                              uint32_t M, uint32_t N, uint32_t K, uint32_t src_rs, uint32_t dst_rs, uint32_t act, float act_p, const float* __restrict__ ctl,
+                              uint32_t M, uint32_t N, uint32_t K, uint32_t src_rs, uint32_t dst_rs, SeqAct act, const float* __restrict__ ctl,
                               uint32_t slot_stride) {
     pdl_enter();
     if (ctl) src += (size_t)ctl_word(ctl, ZG_CTL_SLOT) * slot_stride;      // the rows of a per-sequence state buffer
@@ -53,7 +62,7 @@ __global__ void k_linear_rows(float* __restrict__ dst, const float* __restrict__
     for (int m = 0; m < kGemvRows; m++) {
         if (m < (int)M) {
             const float s = warp_sum(acc[m]);
-            if (lane == 0) dst[(size_t)m * dst_rs + n] = seq_epilogue(s + b, act, act_p);
+            if (lane == 0) dst[(size_t)m * dst_rs + n] = seq_epilogue(s + b, act, n);
         }
     }
 }
@@ -61,7 +70,7 @@ __global__ void k_linear_rows(float* __restrict__ dst, const float* __restrict__
 // vectors per lane are in flight per trip.
 template <typename WT, int MR>
 __global__ void k_linear_rows_vec(float* __restrict__ dst, const float* __restrict__ src, const WT* __restrict__ W, const WT* __restrict__ bias,
-                                  uint32_t M, uint32_t N, uint32_t K, uint32_t src_rs, uint32_t dst_rs, uint32_t act, float act_p, const float* __restrict__ ctl,
+                                  uint32_t M, uint32_t N, uint32_t K, uint32_t src_rs, uint32_t dst_rs, SeqAct act, const float* __restrict__ ctl,
                                   uint32_t slot_stride) {
     // Weights are constants of the model, so this warp's weight row is pulled toward L2 BEFORE the wait on the predecessor:
     // in a replayed graph the HBM stream of a matvec starts under the tail of the kernel that produces its input.
@@ -128,7 +137,7 @@ __global__ void k_linear_rows_vec(float* __restrict__ dst, const float* __restri
     for (int m = 0; m < MR; m++) {
         if (m < (int)M) {
             const float s = warp_sum(acc[m]);
-            if (lane == 0) dst[(size_t)m * dst_rs + n] = seq_epilogue(s + b, act, act_p);
+            if (lane == 0) dst[(size_t)m * dst_rs + n] = seq_epilogue(s + b, act, n);
         }
     }
 }
@@ -138,7 +147,7 @@ constexpr int kTM = 64, kTN = 64, kTK = 16;
 template <typename WT>
 __global__ void __launch_bounds__(256) k_linear_tile(float* __restrict__ dst, const float* __restrict__ src, const WT* __restrict__ W,
                                                      const WT* __restrict__ bias, uint32_t M, uint32_t N, uint32_t K, uint32_t src_rs,
-                                                     uint32_t dst_rs, uint32_t act, float act_p, const float* __restrict__ ctl, uint32_t slot_stride) {
+                                                     uint32_t dst_rs, SeqAct act, const float* __restrict__ ctl, uint32_t slot_stride) {
     __shared__ float As[kTK][kTM + 4];
     __shared__ float Ws[kTK][kTN + 4];
     if (ctl) src += (size_t)ctl_word(ctl, ZG_CTL_SLOT) * slot_stride;
@@ -173,7 +182,7 @@ __global__ void __launch_bounds__(256) k_linear_tile(float* __restrict__ dst, co
 #pragma unroll
         for (int j = 0; j < 4; j++) {
             const uint32_t n = n0 + tx * 4 + j;
-            if (n < N) dst[(size_t)m * dst_rs + n] = seq_epilogue(acc[i][j] + (bias ? wld(bias, n) : 0.0f), act, act_p);
+            if (n < N) dst[(size_t)m * dst_rs + n] = seq_epilogue(acc[i][j] + (bias ? wld(bias, n) : 0.0f), act, n);
         }
     }
 }
@@ -228,6 +237,8 @@ __device__ __forceinline__ float norm_weight(float w, uint32_t kind, float gain)
     if (kind & 2u) w += 1.0f;
     return (kind & 4u) ? w * gain : w;
 }
+// kind bit 5: the weight is a single number for all columns
+__device__ __forceinline__ uint32_t norm_col(uint32_t c, uint32_t kind) { return (kind & 32u) ? 0u : c; }
 template <typename WT>
 __global__ void k_norm(float* __restrict__ dst, const float* __restrict__ src, const WT* __restrict__ w, const float* __restrict__ res,
                        uint32_t cols, uint32_t kind, float eps, float* __restrict__ dst2, const WT* __restrict__ w2, uint32_t kind2, float gain,
@@ -245,8 +256,8 @@ __global__ void k_norm(float* __restrict__ dst, const float* __restrict__ src, c
 #pragma unroll
         for (int i = 0; i < kNormCache; i++) {
             const uint32_t c = threadIdx.x + i * blockDim.x;
-            wa[i] = c < cols ? norm_weight(wld(w, c), kind, gain) : 0.0f;
-            wb[i] = (dst2 && c < cols) ? norm_weight(wld(w2, c), kind2, gain) : 0.0f;
+            wa[i] = c < cols ? norm_weight(wld(w, norm_col(c, kind)), kind, gain) : 0.0f;
+            wb[i] = (dst2 && c < cols) ? norm_weight(wld(w2, norm_col(c, kind2)), kind2, gain) : 0.0f;
         }
     }
     asm volatile("griddepcontrol.wait;" ::: "memory");
@@ -288,10 +299,10 @@ __global__ void k_norm(float* __restrict__ dst, const float* __restrict__ src, c
             __syncthreads();
             x = avg_out + row;
         }
-        norm_pass<false>(dst + row, x, v, res ? res + row : nullptr, rv, cols, kind, eps, sh, false, [&](int, uint32_t c) { return norm_weight(wld(w, c), kind, gain); });
+        norm_pass<false>(dst + row, x, v, res ? res + row : nullptr, rv, cols, kind, eps, sh, false, [&](int, uint32_t c) { return norm_weight(wld(w, norm_col(c, kind)), kind, gain); });
         if (dst2) {
             __syncthreads();                           // the row just written is read back by other threads
-            norm_pass<false>(dst2 + row, dst + row, v, nullptr, rv, cols, kind2, eps, sh, false, [&](int, uint32_t c) { return norm_weight(wld(w2, c), kind2, gain); });
+            norm_pass<false>(dst2 + row, dst + row, v, nullptr, rv, cols, kind2, eps, sh, false, [&](int, uint32_t c) { return norm_weight(wld(w2, norm_col(c, kind2)), kind2, gain); });
         }
     }
     // Single-row steps: the token shift of the launch's last output happens here too.  Every thread revisits the columns it
@@ -340,19 +351,28 @@ __device__ void norm_any_pass(float* out, const float* x, const float* res, cons
     }
     const float alpha = (kind & 8u) ? wld(w, (size_t)2 * cols) : 0.0f;
     for (uint32_t c = threadIdx.x; c < cols; c += blockDim.x) {
-        float y = norm_any_value<WT>(x[c], mean, inv, (kind & 16u) ? 0.0f : wld(w, c), (kind & 8u) ? wld(w, (size_t)cols + c) : 0.0f, kind, gain, alpha);
-        if (xb) y += norm_any_value<WT>(xb[c], mean_b, inv_b, wld(wb, c), 0.0f, kind, gain, 0.0f);
+        float y = norm_any_value<WT>(x[c], mean, inv, (kind & 16u) ? 0.0f : wld(w, norm_col(c, kind)), (kind & 8u) ? wld(w, (size_t)cols + c) : 0.0f, kind, gain, alpha);
+        if (xb) y += norm_any_value<WT>(xb[c], mean_b, inv_b, wld(wb, norm_col(c, kind)), 0.0f, kind, gain, 0.0f);
         out[c] = res ? res[c] + y : y;
     }
+}
+// with an outer norm (w_o) the sum itself is normed once more before it joins the residual.  Every pass touches a column from
+// the same thread, so the second one may run in place.
+template <typename WT>
+__device__ void norm_any_sum(float* out, const float* x, const float* res, const WT* __restrict__ w, uint32_t cols, uint32_t kind, float eps, float gain, float* sh,
+                             const float* xb, const WT* __restrict__ wb, uint32_t kind_o, const WT* __restrict__ w_o) {
+    norm_any_pass(out, x, w_o ? (const float*)nullptr : res, w, cols, kind, eps, gain, sh, xb, wb);
+    if (w_o) norm_any_pass(out, out, res, w_o, cols, kind_o, eps, gain, sh, (const float*)nullptr, (const WT*)nullptr);
 }
 // many rows (prompts): what counts is how many rows are resident per SM, so nothing is kept in registers
 template <typename WT>
 __global__ void __launch_bounds__(256) k_norm_any_rows(float* dst, const float* src, const WT* __restrict__ w, const float* res, uint32_t cols, uint32_t kind, float eps,
-                                                       float* dst2, const WT* __restrict__ w2, uint32_t kind2, float gain, const float* src_b, const WT* __restrict__ w_b) {
+                                                       float* dst2, const WT* __restrict__ w2, uint32_t kind2, float gain, const float* src_b, const WT* __restrict__ w_b,
+                                                       uint32_t kind_o, const WT* __restrict__ w_o) {
     pdl_enter();
     __shared__ float sh[32];
     const size_t row = (size_t)blockIdx.x * cols;
-    norm_any_pass(dst + row, src + row, res ? res + row : nullptr, w, cols, kind, eps, gain, sh, src_b ? src_b + row : nullptr, w_b);
+    norm_any_sum(dst + row, src + row, res ? res + row : nullptr, w, cols, kind, eps, gain, sh, src_b ? src_b + row : nullptr, w_b, kind_o, w_o);
     if (dst2) {
         __syncthreads();                                   // the row just written is read back by other threads
         norm_any_pass(dst2 + row, dst + row, (const float*)nullptr, w2, cols, kind2, eps, gain, sh, (const float*)nullptr, (const WT*)nullptr);
@@ -360,27 +380,29 @@ __global__ void __launch_bounds__(256) k_norm_any_rows(float* dst, const float* 
 }
 template <typename WT, int kKeep, int kThreads>          // a row of up to kKeep x kThreads values lives in registers (fewer kept values, more CTAs per SM)
 __global__ void __launch_bounds__(kThreads) k_norm_any(float* dst, const float* src, const WT* __restrict__ w, const float* res, uint32_t cols, uint32_t kind, float eps,
-                                                  float* dst2, const WT* __restrict__ w2, uint32_t kind2, float gain, const float* src_b, const WT* __restrict__ w_b) {
+                                                  float* dst2, const WT* __restrict__ w2, uint32_t kind2, float gain, const float* src_b, const WT* __restrict__ w_b,
+                                                       uint32_t kind_o, const WT* __restrict__ w_o) {
     asm volatile("griddepcontrol.launch_dependents;" ::: "memory");
     __shared__ float sh[32];
     const size_t row = (size_t)blockIdx.x * cols;
     if (cols > kKeep * kThreads) {                  // rows too wide for the registers
         asm volatile("griddepcontrol.wait;" ::: "memory");
-        norm_any_pass(dst + row, src + row, res ? res + row : nullptr, w, cols, kind, eps, gain, sh, src_b ? src_b + row : nullptr, w_b);
+        norm_any_sum(dst + row, src + row, res ? res + row : nullptr, w, cols, kind, eps, gain, sh, src_b ? src_b + row : nullptr, w_b, kind_o, w_o);
         if (dst2) {
             __syncthreads();                               // the row just written is read back by other threads
             norm_any_pass(dst2 + row, dst + row, (const float*)nullptr, w2, cols, kind2, eps, gain, sh, (const float*)nullptr, (const WT*)nullptr);
         }
         return;
     }
-    float v[kKeep], wa[kKeep], aux[kKeep], wc[kKeep], bc[kKeep];   // aux: the bias of a Dynamic Tanh, or the second source's weight
+    float v[kKeep], wa[kKeep], aux[kKeep], wc[kKeep], bc[kKeep], wo[kKeep];   // aux: the bias of a Dynamic Tanh, or the second source's weight
 #pragma unroll
     for (int i = 0; i < kKeep; i++) {
         const uint32_t c = threadIdx.x + i * blockDim.x;
         const bool in = c < cols;
-        wa[i] = (in && !(kind & 16u)) ? wld(w, c) : 0.0f;
-        aux[i] = in ? ((kind & 8u) ? wld(w, (size_t)cols + c) : (src_b ? wld(w_b, c) : 0.0f)) : 0.0f;
-        wc[i] = (in && dst2 && !(kind2 & 16u)) ? wld(w2, c) : 0.0f;
+        wa[i] = (in && !(kind & 16u)) ? wld(w, norm_col(c, kind)) : 0.0f;
+        aux[i] = in ? ((kind & 8u) ? wld(w, (size_t)cols + c) : (src_b ? wld(w_b, norm_col(c, kind)) : 0.0f)) : 0.0f;
+        wc[i] = (in && dst2 && !(kind2 & 16u)) ? wld(w2, norm_col(c, kind2)) : 0.0f;
+        wo[i] = (in && w_o) ? wld(w_o, norm_col(c, kind_o)) : 0.0f;
         bc[i] = (in && dst2 && (kind2 & 8u)) ? wld(w2, (size_t)cols + c) : 0.0f;
     }
     const float alpha = (kind & 8u) ? wld(w, (size_t)2 * cols) : 0.0f, alpha2 = (dst2 && (kind2 & 8u)) ? wld(w2, (size_t)2 * cols) : 0.0f;
@@ -416,10 +438,22 @@ __global__ void __launch_bounds__(kThreads) k_norm_any(float* dst, const float* 
 #pragma unroll
     for (int i = 0; i < kKeep; i++) {
         const uint32_t c = threadIdx.x + i * blockDim.x;
+        if (c >= cols) { v[i] = 0.0f; continue; }       // columns past the row stay zero (a layer norm would shift them)
         float y = norm_any_value<WT>(v[i], mean, inv, wa[i], aux[i], kind, gain, alpha);
         if (src_b) y += norm_any_value<WT>(vb[i], mean_b, inv_b, aux[i], 0.0f, kind, gain, 0.0f);
+        if (w_o) { v[i] = y; continue; }
         v[i] = res ? rv[i] + y : y;
         if (c < cols) dst[row + c] = v[i];
+    }
+    if (w_o) {                                      // the sum is normed once more before it joins the residual
+        stats(v, kind_o, mean, inv);
+#pragma unroll
+        for (int i = 0; i < kKeep; i++) {
+            const uint32_t c = threadIdx.x + i * blockDim.x;
+            const float y = norm_any_value<WT>(v[i], mean, inv, wo[i], 0.0f, kind_o, gain, 0.0f);
+            v[i] = res ? rv[i] + y : y;
+            if (c < cols) dst[row + c] = v[i];
+        }
     }
     if (!dst2) return;
     stats(v, kind2, mean, inv);
@@ -850,8 +884,8 @@ __global__ void k_conv_advance(float* __restrict__ state, const float* __restric
 // prepared by the whole CTA at once, then the tokens are walked without further barriers.
 constexpr int kDeltaRows = 16, kDeltaTile = 16, kDeltaThreads = 128;
 // forms of the rule (op parameter n10): plain accumulation without unit vectors and correction (gated linear attention), the
-// decay as a tempered sigmoid, a SiLU output gate, an output scale
-constexpr uint32_t kDeltaPlain = 1, kDeltaSigmoidDecay = 2, kDeltaSiluGate = 4, kDeltaOutScale = 8;
+// decay as a tempered sigmoid, a SiLU output gate, an output scale, one decay per head instead of one per key channel
+constexpr uint32_t kDeltaPlain = 1, kDeltaSigmoidDecay = 2, kDeltaSiluGate = 4, kDeltaOutScale = 8, kDeltaHeadDecay = 16;
 // decay of one key channel from its logit z (the bias is already added): exp(-exp(A) softplus(z)), or sigmoid(z)^(1 / tau) =
 // exp(-softplus(-z) / tau)
 __device__ __forceinline__ float delta_decay(float z, float Ah, uint32_t form, float inv_tau) {
@@ -866,6 +900,7 @@ __global__ void __launch_bounds__(kDeltaThreads) k_delta_rule(
     pdl_enter();
     extern __shared__ float sm[];
     const bool plain = form & kDeltaPlain;             // no unit vectors, no correction: S <- g S + k v^T
+    const bool head_decay = form & kDeltaHeadDecay;    // a row of `ab` holds one logit per head
     const uint32_t dpad = RS * kDeltaRows;             // rows incl. padding (k = q = 0, decay = 1 there)
     float* sk = sm;                                    // [tile][dpad]
     float* sq = sk + kDeltaTile * dpad;
@@ -893,7 +928,8 @@ __global__ void __launch_bounds__(kDeltaThreads) k_delta_rule(
             const uint32_t t = t0 + tt;
             const float* qr = qkv + (size_t)t * qkv_rs + q_off + (size_t)kv * dim;
             const float* kr = qkv + (size_t)t * qkv_rs + k_off + (size_t)kv * dim;
-            const float* ar = ab + (size_t)t * a_rs + (size_t)h * dim;
+            const float* ar = ab + (size_t)t * a_rs + (head_decay ? (size_t)h : (size_t)h * dim);
+            const float gh = head_decay ? delta_decay(ar[0] + wld(wts, (size_t)dt_off + h), Ah, form, inv_tau) : 1.0f;
             float qn = q_scale, kn = 1.0f;
             if (!plain) {
                 float qq = 0.0f, kk = 0.0f;
@@ -904,7 +940,7 @@ __global__ void __launch_bounds__(kDeltaThreads) k_delta_rule(
                 const bool in = c < dim;
                 sk[tt * dpad + c] = in ? kr[c] * kn : 0.0f;
                 sq[tt * dpad + c] = in ? qr[c] * qn : 0.0f;
-                sg[tt * dpad + c] = in ? delta_decay(ar[c] + wld(wts, (size_t)dt_off + (size_t)h * dim + c), Ah, form, inv_tau) : 1.0f;
+                sg[tt * dpad + c] = head_decay ? gh : in ? delta_decay(ar[c] + wld(wts, (size_t)dt_off + (size_t)h * dim + c), Ah, form, inv_tau) : 1.0f;
             }
             if (lane == 0) sbeta[tt] = plain ? 1.0f : sigmoidf_(betab[(size_t)t * beta_rs + beta_off + h]);
         }
@@ -966,38 +1002,41 @@ __global__ void k_delta_prepare(float* __restrict__ prep, const float* __restric
                                 uint32_t k_off, uint32_t beta_off, uint32_t A_off, uint32_t dt_off, uint32_t qkv_rs, uint32_t beta_rs, uint32_t a_rs,
                                 float unit_eps, float q_scale, uint32_t form, float inv_tau) {
     pdl_enter();
-    const bool plain = form & kDeltaPlain;
+    const bool plain = form & kDeltaPlain, head_decay = form & kDeltaHeadDecay;
     const uint32_t w = blockIdx.x * (blockDim.x >> 5) + (threadIdx.x >> 5), lane = threadIdx.x & 31;
     if (w >= T * H) return;
     const uint32_t t = w / H, h = w % H, kv = h / (H / G);
     const float* qr = qkv + (size_t)t * qkv_rs + q_off + (size_t)kv * dim;
     const float* kr = qkv + (size_t)t * qkv_rs + k_off + (size_t)kv * dim;
-    const float* ar = ab + (size_t)t * a_rs + (size_t)h * dim;
+    const float* ar = ab + (size_t)t * a_rs + (head_decay ? (size_t)h : (size_t)h * dim);
     float qq = 0.0f, kk = 0.0f, qk = 0.0f;
     for (uint32_t c = lane; c < dim; c += 32) { const float a = qr[c], b = kr[c]; qq = fmaf(a, a, qq); kk = fmaf(b, b, kk); qk = fmaf(a, b, qk); }
     const float qn = plain ? q_scale : q_scale / sqrtf(warp_sum(qq) + unit_eps), kn = plain ? 1.0f : 1.0f / sqrtf(warp_sum(kk) + unit_eps);
     qk = warp_sum(qk) * qn * kn;
     const float Ah = (form & kDeltaSigmoidDecay) ? 0.0f : expf(wld(wts, (size_t)A_off + h));
-    float* row = prep + ((size_t)h * T + t) * (3 * dpad + 4);
+    float* row = prep + ((size_t)h * T + t) * ((head_decay ? 2 : 3) * dpad + 4);
+    const float gh = head_decay ? delta_decay(ar[0] + wld(wts, (size_t)dt_off + h), Ah, form, inv_tau) : 0.0f;
     for (uint32_t c = lane; c < dpad; c += 32) {
         const bool in = c < dim;
         row[c] = in ? kr[c] * kn : 0.0f;
         row[dpad + c] = in ? qr[c] * qn : 0.0f;
-        row[2 * dpad + c] = in ? delta_decay(ar[c] + wld(wts, (size_t)dt_off + (size_t)h * dim + c), Ah, form, inv_tau) : 1.0f;
+        if (!head_decay) row[2 * dpad + c] = in ? delta_decay(ar[c] + wld(wts, (size_t)dt_off + (size_t)h * dim + c), Ah, form, inv_tau) : 1.0f;
     }
-    if (lane < 4) row[3 * dpad + lane] = lane == 0 ? (plain ? 1.0f : sigmoidf_(betab[(size_t)t * beta_rs + beta_off + h])) : (lane == 1 ? qk : 0.0f);
+    if (lane < 4) row[(head_decay ? 2 : 3) * dpad + lane] = lane == 0 ? (plain ? 1.0f : sigmoidf_(betab[(size_t)t * beta_rs + beta_off + h])) : (lane == 1 ? qk : (lane == 2 ? gh : 0.0f));
 }
 __device__ __forceinline__ void cp_async16(float* smem_dst, const float* gmem_src) {
     asm volatile("cp.async.cg.shared.global [%0], [%1], 16;" ::"r"((uint32_t)__cvta_generic_to_shared(smem_dst)), "l"(gmem_src) : "memory");
 }
 // PLAIN: the accumulation without correction (u = v), which needs no product with k and only one reduction per token
-template <uint32_t RS, bool PLAIN>                     // row slices of a column: compile-time, so the shuffle steps unroll
+// HEADG: one decay per head and token.  It commutes with the sums over the key rows, so both dot products run on the state as
+// the token finds it and the decay joins the two results: u = beta (v - g S^T k), o = g S^T q + u (k . q), S <- g S + k u^T.
+template <uint32_t RS, bool PLAIN, bool HEADG>                     // row slices of a column: compile-time, so the shuffle steps unroll
 __global__ void __launch_bounds__(kWalkThreads) k_delta_walk(float* __restrict__ dst, const float* __restrict__ qkv, const float* __restrict__ prep,
                                                                float* __restrict__ state, const float* __restrict__ ctl, uint32_t T, uint32_t H,
                                                                uint32_t dim, uint32_t vdim, uint32_t v_off, uint32_t qkv_rs, uint32_t dst_rs) {
     pdl_enter();
     extern __shared__ __align__(16) float sm[];
-    const uint32_t dpad = RS * kWalkRows, stride = 3 * dpad + 4, tile_elems = kDeltaTile * stride;
+    const uint32_t dpad = RS * kWalkRows, tail = (HEADG ? 2 : 3) * dpad, stride = tail + 4, tile_elems = kDeltaTile * stride;
     const uint32_t h = blockIdx.y;
     const uint32_t cols_per_cta = kWalkThreads / RS;
     const uint32_t r = threadIdx.x % RS, col = blockIdx.x * cols_per_cta + threadIdx.x / RS;
@@ -1036,7 +1075,8 @@ __global__ void __launch_bounds__(kWalkThreads) k_delta_walk(float* __restrict__
         const float* tile = sm + cur * tile_elems;
         auto token = [&](int tti, float v) {
             const float* row = tile + tti * stride;
-            const float beta = row[3 * dpad], kq = row[3 * dpad + 1];   // read with the vectors, before the shuffles
+            const float4 tl = *reinterpret_cast<const float4*>(row + tail);   // beta, k . q, the head's decay: read with the vectors, before the shuffles
+            const float beta = tl.x, kq = tl.y, gh = tl.z;
             float4 k4[kWalkRows / 4], g4[kWalkRows / 4];
             float ks0 = 0.0f, ks1 = 0.0f, qs0 = 0.0f, qs1 = 0.0f;
 #pragma unroll
@@ -1044,8 +1084,10 @@ __global__ void __launch_bounds__(kWalkThreads) k_delta_walk(float* __restrict__
                 const uint32_t at = (c * RS + r) * 4;
                 k4[c] = *reinterpret_cast<const float4*>(row + at);
                 const float4 q4 = *reinterpret_cast<const float4*>(row + dpad + at);
-                g4[c] = *reinterpret_cast<const float4*>(row + 2 * dpad + at);
-                S[4 * c + 0] *= g4[c].x; S[4 * c + 1] *= g4[c].y; S[4 * c + 2] *= g4[c].z; S[4 * c + 3] *= g4[c].w;
+                if (!HEADG) {
+                    g4[c] = *reinterpret_cast<const float4*>(row + 2 * dpad + at);
+                    S[4 * c + 0] *= g4[c].x; S[4 * c + 1] *= g4[c].y; S[4 * c + 2] *= g4[c].z; S[4 * c + 3] *= g4[c].w;
+                }
                 if (!PLAIN) {
                     ks0 = fmaf(S[4 * c + 0], k4[c].x, ks0); ks1 = fmaf(S[4 * c + 1], k4[c].y, ks1);
                     ks0 = fmaf(S[4 * c + 2], k4[c].z, ks0); ks1 = fmaf(S[4 * c + 3], k4[c].w, ks1);
@@ -1056,9 +1098,11 @@ __global__ void __launch_bounds__(kWalkThreads) k_delta_walk(float* __restrict__
             float ks = ks0 + ks1, qs = qs0 + qs1;
 #pragma unroll
             for (uint32_t o = 1; o < RS; o <<= 1) { if (!PLAIN) ks += __shfl_xor_sync(0xffffffffu, ks, o); qs += __shfl_xor_sync(0xffffffffu, qs, o); }
+            if (HEADG) { ks *= gh; qs *= gh; }
             const float u = PLAIN ? v : beta * (v - ks);
 #pragma unroll
             for (int c = 0; c < kWalkRows / 4; c++) {
+                if (HEADG) { S[4 * c + 0] *= gh; S[4 * c + 1] *= gh; S[4 * c + 2] *= gh; S[4 * c + 3] *= gh; }
                 S[4 * c + 0] = fmaf(k4[c].x, u, S[4 * c + 0]); S[4 * c + 1] = fmaf(k4[c].y, u, S[4 * c + 1]);
                 S[4 * c + 2] = fmaf(k4[c].z, u, S[4 * c + 2]); S[4 * c + 3] = fmaf(k4[c].w, u, S[4 * c + 3]);
             }
@@ -1431,6 +1475,7 @@ bool zg_seq_op_valid(const ZgOp& op, const size_t* elems, size_t n_bufs, char* w
         case ZG_OP_EMBED: {
             const size_t T = s.n[0], D = s.n[1];
             if (!fits(0, 0, T * D) || !fits(1, ZG_CTL_IDS, T) || !have(2)) return fail("embed: extent");
+            if (s.n[4] && (s.n[3] || s.n[5] >= s.n[4] || s.n[6] >= s.n[4] || !wfits(2, s.off[2], ((size_t)s.n[4] + 1) * D))) return fail("embed: bigram table");
             return true;
         }
         case ZG_OP_LINEAR: {
@@ -1439,20 +1484,28 @@ bool zg_seq_op_valid(const ZgOp& op, const size_t* elems, size_t n_bufs, char* w
             if (!fits(0, s.off[3], (M - 1) * drs + N) || !fits(1, s.off[2], (M - 1) * srs + K) || !wfits(2, s.off[0], N * K)) return fail("linear: extent");
             if (s.buf[3] != ZG_NO_BUF && !wfits(3, s.off[1], N)) return fail("linear: bias extent");
             if (s.buf[0] == s.buf[1]) return fail("linear: in place");
-            if (s.n[6] > 5 || (s.n[6] == 5 && !(s.f[0] > 0.0f))) return fail("linear: activation");
+            if (s.n[6] > 6 || (s.n[6] == 5 && !(s.f[0] > 0.0f))) return fail("linear: activation");
+            if (s.n[9] > N || s.n[8] > (s.n[9] ? s.n[9] : N)) return fail("linear: activation columns");
             if (s.n[7] && (s.n[7] < s.off[2] + (M - 1) * srs + K || !fits(4, 0, ZG_CTL_IDS))) return fail("linear: source slots");
             return true;
         }
         case ZG_OP_NORM: {
             const size_t n = (size_t)s.n[0] * s.n[1];
-            if (!n || s.n[2] > 31 || (s.n[2] & 24u) == 24u) return fail("norm: shape");
-            const size_t w_need = (s.n[2] & 8u) ? 2 * (size_t)s.n[1] + 1 : s.n[1];      // Dynamic Tanh: weight, bias and alpha
+            auto bad_kind = [](uint32_t k) { return k > 63 || (k & 24u) == 24u || ((k & 32u) && (k & 24u)); };
+            auto weights = [&](uint32_t k) { return (k & 8u) ? 2 * (size_t)s.n[1] + 1 : ((k & 32u) ? (size_t)1 : (size_t)s.n[1]); };
+            if (!n || bad_kind(s.n[2])) return fail("norm: shape");
+            const size_t w_need = weights(s.n[2]);      // Dynamic Tanh: weight, bias and alpha
             if (!fits(0, s.off[3], n) || !fits(1, 0, n) || (!(s.n[2] & 16u) && !wfits(2, s.off[0], w_need))) return fail("norm: extent");
             if (s.n[7]) {      // a second source, normed like the first with its own weight (off 2 of w's arena) and added to it
-                if (s.n[7] > 1 || (s.n[2] & 24u) || s.n[5] || !fits(6, 0, n) || !wfits(2, s.off[2], s.n[1]) || s.buf[6] == s.buf[0] || (s.buf[4] != ZG_NO_BUF && s.buf[6] == s.buf[4]))
+                if (s.n[7] > 1 || (s.n[2] & 24u) || s.n[5] || !fits(6, 0, n) || !wfits(2, s.off[2], w_need) || s.buf[6] == s.buf[0] || (s.buf[4] != ZG_NO_BUF && s.buf[6] == s.buf[4]))
                     return fail("norm: second source");
             } else if (((s.n[2] | (s.buf[4] != ZG_NO_BUF && !s.n[5] ? s.n[4] : 0u)) & 24u) && (s.n[5] || s.buf[6] != ZG_NO_BUF))
                 return fail("norm: kinds without statistics take no averaged source and no token shift");
+            if (s.n[8]) {      // an outer norm over the (sum of the) normed source(s)
+                const uint32_t ko = s.n[8] - 1;
+                if (bad_kind(ko) || (ko & 28u) || (s.n[2] & 24u) || s.n[5] || (!s.n[7] && s.buf[6] != ZG_NO_BUF) || !wfits(2, s.off[5], weights(ko)) || s.buf[0] == s.buf[3])
+                    return fail("norm: outer norm");
+            }
             if (s.n[5]) {      // averaged source
                 if (s.n[6] < n || !fits(1, 0, (size_t)(s.n[5] - 1) * s.n[6] + n) || !wfits(2, s.off[4], s.n[5]) || s.buf[3] != ZG_NO_BUF || !fits(4, 0, n) || s.buf[4] == s.buf[0] ||
                     s.buf[4] == s.buf[1])
@@ -1461,7 +1514,7 @@ bool zg_seq_op_valid(const ZgOp& op, const size_t* elems, size_t n_bufs, char* w
                 return true;
             }
             if (s.buf[3] != ZG_NO_BUF && !fits(3, 0, n)) return fail("norm: residual extent");
-            if (s.buf[4] != ZG_NO_BUF && (s.n[4] > 31 || (s.n[4] & 24u) == 24u || !fits(4, 0, n) || (!(s.n[4] & 16u) && !wfits(5, s.off[1], (s.n[4] & 8u) ? 2 * (size_t)s.n[1] + 1 : s.n[1])) || s.buf[4] == s.buf[0] || s.buf[4] == s.buf[1] || s.buf[4] == s.buf[3]))
+            if (s.buf[4] != ZG_NO_BUF && (bad_kind(s.n[4]) || !fits(4, 0, n) || (!(s.n[4] & 16u) && !wfits(5, s.off[1], weights(s.n[4]))) || s.buf[4] == s.buf[0] || s.buf[4] == s.buf[1] || s.buf[4] == s.buf[3]))
                 return fail("norm: chained norm");
             if (!s.n[7] && s.buf[6] != ZG_NO_BUF && (s.n[0] != 1 || !have(6) || elems[s.buf[6]] < s.n[1] || !wfits(s.buf[4] != ZG_NO_BUF ? 5 : 2, s.off[2], s.n[1]) || !fits(7, 0, ZG_CTL_IDS)))
                 return fail("norm: fused token shift (single-row steps)");
@@ -1488,12 +1541,12 @@ bool zg_seq_op_valid(const ZgOp& op, const size_t* elems, size_t n_bufs, char* w
         case ZG_OP_DELTA_RULE: {
             const size_t T = s.n[0], H = s.n[1], G = s.n[2], dim = s.n[3], vdim = s.n[4];
             const size_t form = s.n[10], drs = s.n[11] ? s.n[11] : H * vdim;
-            if (!T || !H || !G || H % G || !dim || !vdim || zg_delta_row_slices((uint32_t)dim) > 32 || form > 15) return fail("delta_rule: shape");
+            if (!T || !H || !G || H % G || !dim || !vdim || zg_delta_row_slices((uint32_t)dim) > 32 || form > 31) return fail("delta_rule: shape");
             if (s.n[12] + H * vdim > drs || ((form & 2) && !(s.f[3] > 0.0f))) return fail("delta_rule: form");
-            if (s.off[0] + G * dim > s.n[5] || s.off[1] + G * dim > s.n[5] || s.off[2] + H * vdim > s.n[5] || (!(form & 1) && s.off[3] + H > s.n[6]) || H * dim > s.n[7] || s.off[7] + H * vdim > s.n[8])
+            if (s.off[0] + G * dim > s.n[5] || s.off[1] + G * dim > s.n[5] || s.off[2] + H * vdim > s.n[5] || (!(form & 1) && s.off[3] + H > s.n[6]) || s.n[13] + H * (form & 16 ? 1 : dim) > s.n[7] || s.off[7] + H * vdim > s.n[8])
                 return fail("delta_rule: columns");
             if (!fits(0, 0, (T - 1) * drs + s.n[12] + H * vdim) || !fits(1, 0, T * s.n[5]) || (!(form & 1) && !fits(2, 0, T * s.n[6])) || !fits(3, 0, T * s.n[7]) || !fits(4, 0, T * s.n[8]) ||
-                (!(form & 2) && !wfits(5, s.off[4], H)) || !wfits(5, s.off[5], H * dim) || !wfits(5, s.off[6], vdim) || !have(6) || elems[s.buf[6]] < H * dim * vdim || !fits(7, 0, ZG_CTL_IDS))
+                (!(form & 2) && !wfits(5, s.off[4], H)) || !wfits(5, s.off[5], H * (form & 16 ? 1 : dim)) || !wfits(5, s.off[6], vdim) || !have(6) || elems[s.buf[6]] < H * dim * vdim || !fits(7, 0, ZG_CTL_IDS))
                 return fail("delta_rule: extent");
             return true;
         }
@@ -1548,7 +1601,7 @@ size_t zg_seq_op_scratch_elems(const ZgOp& op, float* const* bufs) {
     }
     if (op.tag == ZG_OP_DELTA_RULE) {                  // the prepared per-token rows of the prefill form
         const ZgSeqOp& d = op.u.seq;
-        return d.n[0] >= (uint32_t)kDeltaPrepMinTokens && d.n[3] <= (uint32_t)kWalkMaxDim ? (size_t)d.n[0] * d.n[1] * (3 * delta_walk_slices(d.n[3]) * kWalkRows + 4) : 0;
+        return d.n[0] >= (uint32_t)kDeltaPrepMinTokens && d.n[3] <= (uint32_t)kWalkMaxDim ? (size_t)d.n[0] * d.n[1] * ((d.n[10] & kDeltaHeadDecay ? 2 : 3) * delta_walk_slices(d.n[3]) * kWalkRows + 4) : 0;
     }
     if (!dense_gemm_enabled() || op.tag != ZG_OP_LINEAR || op.u.seq.n[5] != ZG_W_BF16) return 0;
     const ZgSeqOp& s = op.u.seq;
@@ -1562,7 +1615,7 @@ bool zg_launch_seq_op(ZgCudaCtx* ctx, const ZgOp& op, float* const* bufs, float*
     switch (op.tag) {
         case ZG_OP_EMBED:
             ZG_SEQ_WDT(s.n[2], launch_pdl(k_embed<WT>, dim3(s.n[0]), dim3(128), 0, st, bufs[s.buf[0]], bufs[s.buf[1]], wptr<WT>(bufs, s.buf[2], s.off[0]), s.n[1], s.f[0],
-                                          s.n[3] ? wptr<WT>(bufs, s.buf[2], s.off[1]) : nullptr));
+                                          s.n[3] ? wptr<WT>(bufs, s.buf[2], s.off[1]) : nullptr, s.n[4] ? wptr<WT>(bufs, s.buf[2], s.off[2]) : nullptr, s.n[4], s.n[5], s.n[6]));
             ZG_SEQ_CHECK();
             return true;
         case ZG_OP_LINEAR: {
@@ -1570,10 +1623,11 @@ bool zg_launch_seq_op(ZgCudaCtx* ctx, const ZgOp& op, float* const* bufs, float*
             float* dst = bufs[s.buf[0]] + s.off[3];
             const float* src = bufs[s.buf[1]] + s.off[2];
             const bool has_bias = s.buf[3] != ZG_NO_BUF;
+            const SeqAct act = {s.n[6], s.f[0], s.n[8], s.n[9] ? s.n[9] : N};
             const float* slot_ctl = s.n[7] ? (const float*)bufs[s.buf[4]] : (const float*)nullptr;      // the source is the slot's part of a state buffer
             if (scratch && zg_seq_op_scratch_elems(op, bufs))
                 return zg_dense_gemm_launch(wptr<bf16>(bufs, s.buf[2], s.off[0]), has_bias ? wptr<bf16>(bufs, s.buf[3], s.off[1]) : nullptr, src, dst, M, N, K,
-                                            s.n[3], s.n[4], scratch, st, s.n[6], s.f[0], slot_ctl, s.n[7]);
+                                            s.n[3], s.n[4], scratch, st, s.n[6], s.f[0], act.lo, act.hi, slot_ctl, s.n[7]);
             ZG_SEQ_WDT(s.n[5], {
                 const WT* W = wptr<WT>(bufs, s.buf[2], s.off[0]);
                 const WT* b = has_bias ? wptr<WT>(bufs, s.buf[3], s.off[1]) : nullptr;
@@ -1582,13 +1636,13 @@ bool zg_launch_seq_op(ZgCudaCtx* ctx, const ZgOp& op, float* const* bufs, float*
                     const size_t xs_bytes = (size_t)M * K * sizeof(float);
                     const bool vec = K % V == 0 && (reinterpret_cast<size_t>(W) & 15) == 0 && xs_bytes <= 48 * 1024;
                     const dim3 grid((N + 7) / 8);
-                    if (vec && M == 1) launch_pdl(k_linear_rows_vec<WT, 1>, dim3(grid), dim3(256), xs_bytes, st, dst, src, W, b, M, N, K, s.n[3], s.n[4], s.n[6], s.f[0], slot_ctl, s.n[7]);
-                    else if (vec && M <= 4) launch_pdl(k_linear_rows_vec<WT, 4>, dim3(grid), dim3(256), xs_bytes, st, dst, src, W, b, M, N, K, s.n[3], s.n[4], s.n[6], s.f[0], slot_ctl, s.n[7]);
-                    else if (vec) launch_pdl(k_linear_rows_vec<WT, 8>, dim3(grid), dim3(256), xs_bytes, st, dst, src, W, b, M, N, K, s.n[3], s.n[4], s.n[6], s.f[0], slot_ctl, s.n[7]);
-                    else launch_pdl(k_linear_rows<WT>, dim3(grid), dim3(256), 0, st, dst, src, W, b, M, N, K, s.n[3], s.n[4], s.n[6], s.f[0], slot_ctl, s.n[7]);
+                    if (vec && M == 1) launch_pdl(k_linear_rows_vec<WT, 1>, dim3(grid), dim3(256), xs_bytes, st, dst, src, W, b, M, N, K, s.n[3], s.n[4], act, slot_ctl, s.n[7]);
+                    else if (vec && M <= 4) launch_pdl(k_linear_rows_vec<WT, 4>, dim3(grid), dim3(256), xs_bytes, st, dst, src, W, b, M, N, K, s.n[3], s.n[4], act, slot_ctl, s.n[7]);
+                    else if (vec) launch_pdl(k_linear_rows_vec<WT, 8>, dim3(grid), dim3(256), xs_bytes, st, dst, src, W, b, M, N, K, s.n[3], s.n[4], act, slot_ctl, s.n[7]);
+                    else launch_pdl(k_linear_rows<WT>, dim3(grid), dim3(256), 0, st, dst, src, W, b, M, N, K, s.n[3], s.n[4], act, slot_ctl, s.n[7]);
                 } else {
                     const dim3 grid((N + kTN - 1) / kTN, (M + kTM - 1) / kTM);
-                    k_linear_tile<WT><<<grid, 256, 0, st>>>(dst, src, W, b, M, N, K, s.n[3], s.n[4], s.n[6], s.f[0], slot_ctl, s.n[7]);
+                    k_linear_tile<WT><<<grid, 256, 0, st>>>(dst, src, W, b, M, N, K, s.n[3], s.n[4], act, slot_ctl, s.n[7]);
                 }
             });
             ZG_SEQ_CHECK();
@@ -1599,17 +1653,19 @@ bool zg_launch_seq_op(ZgCudaCtx* ctx, const ZgOp& op, float* const* bufs, float*
             float* dst2 = s.buf[4] != ZG_NO_BUF ? bufs[s.buf[4]] : nullptr;
             float* shift_state = s.buf[6] != ZG_NO_BUF ? bufs[s.buf[6]] : nullptr;
             const uint32_t avg_terms = s.n[5];             // averaged source: buf 4 receives the average instead of a chained norm
-            if (((s.n[2] | (dst2 ? s.n[4] : 0u)) & 24u) || s.n[7]) {   // Dynamic Tanh or the plain residual step somewhere in the launch, or two sources
+            if (((s.n[2] | (dst2 ? s.n[4] : 0u)) & 24u) || s.n[7] || s.n[8]) {   // Dynamic Tanh or the plain residual step somewhere in the launch, or two sources
 #define ZG_NORM_ANY(KEEP_, THREADS_)                                                                                                               \
     ZG_SEQ_WDT(s.n[3], launch_pdl(k_norm_any<WT, KEEP_, THREADS_>, dim3(s.n[0]), dim3(THREADS_), 0, st, bufs[s.buf[0]] + s.off[3], (const float*)bufs[s.buf[1]], \
                                   (s.n[2] & 16u) ? (const WT*)nullptr : wptr<WT>(bufs, s.buf[2], s.off[0]), res, s.n[1], s.n[2], s.f[0], dst2,                \
                                   dst2 && !(s.n[4] & 16u) ? wptr<WT>(bufs, s.buf[5], s.off[1]) : (const WT*)nullptr, s.n[4], s.f[1],                         \
-                                  s.n[7] ? (const float*)bufs[s.buf[6]] : (const float*)nullptr, s.n[7] ? wptr<WT>(bufs, s.buf[2], s.off[2]) : (const WT*)nullptr))
+                                  s.n[7] ? (const float*)bufs[s.buf[6]] : (const float*)nullptr, s.n[7] ? wptr<WT>(bufs, s.buf[2], s.off[2]) : (const WT*)nullptr, \
+                                  s.n[8] ? s.n[8] - 1 : 0u, s.n[8] ? wptr<WT>(bufs, s.buf[2], s.off[5]) : (const WT*)nullptr))
                 if (s.n[0] >= 64 || s.n[1] > 4096)
                     ZG_SEQ_WDT(s.n[3], launch_pdl(k_norm_any_rows<WT>, dim3(s.n[0]), dim3(256), 0, st, bufs[s.buf[0]] + s.off[3], (const float*)bufs[s.buf[1]],
                                                   (s.n[2] & 16u) ? (const WT*)nullptr : wptr<WT>(bufs, s.buf[2], s.off[0]), res, s.n[1], s.n[2], s.f[0], dst2,
                                                   dst2 && !(s.n[4] & 16u) ? wptr<WT>(bufs, s.buf[5], s.off[1]) : (const WT*)nullptr, s.n[4], s.f[1],
-                                                  s.n[7] ? (const float*)bufs[s.buf[6]] : (const float*)nullptr, s.n[7] ? wptr<WT>(bufs, s.buf[2], s.off[2]) : (const WT*)nullptr));
+                                                  s.n[7] ? (const float*)bufs[s.buf[6]] : (const float*)nullptr, s.n[7] ? wptr<WT>(bufs, s.buf[2], s.off[2]) : (const WT*)nullptr,
+                                                  s.n[8] ? s.n[8] - 1 : 0u, s.n[8] ? wptr<WT>(bufs, s.buf[2], s.off[5]) : (const WT*)nullptr));
                 else if (s.n[1] <= 1024) ZG_NORM_ANY(4, 256);
                 else if (s.n[1] <= 2048) ZG_NORM_ANY(8, 256);
                 else ZG_NORM_ANY(8, 512);                      // up to 4096 columns in registers; wider rows are walked from memory
@@ -1695,28 +1751,29 @@ bool zg_launch_seq_op(ZgCudaCtx* ctx, const ZgOp& op, float* const* bufs, float*
             const dim3 grid((vdim + cols - 1) / cols, H);
             if (scratch && T >= (uint32_t)kDeltaPrepMinTokens && dim <= (uint32_t)kWalkMaxDim) {
                 const uint32_t WS = delta_walk_slices(dim), dpad = WS * kWalkRows, wcols = kWalkThreads / WS;
-                const size_t walk_smem = (size_t)2 * kDeltaTile * (3 * dpad + 4) * sizeof(float);
-                ZG_SEQ_WDT(s.n[9], launch_pdl(k_delta_prepare<WT>, dim3((T * H + 3) / 4), dim3(128), 0, st, scratch, bufs[s.buf[1]], betab, bufs[s.buf[3]],
+                const size_t walk_smem = (size_t)2 * kDeltaTile * ((form & kDeltaHeadDecay ? 2 : 3) * dpad + 4) * sizeof(float);
+                ZG_SEQ_WDT(s.n[9], launch_pdl(k_delta_prepare<WT>, dim3((T * H + 3) / 4), dim3(128), 0, st, scratch, bufs[s.buf[1]], betab, bufs[s.buf[3]] + s.n[13],
                                               wptr<WT>(bufs, s.buf[5], 0), T, H, G, dim, dpad, s.off[0], s.off[1], s.off[3], s.off[4], s.off[5], s.n[5], s.n[6], s.n[7], s.f[1], s.f[2],
                                               form, inv_tau));
                 ZG_SEQ_CHECK();
+#define ZG_WALK_FORM(RS_, PLAIN_, HEADG_)                                                                                                       \
+    do {                                                                                                                                        \
+        if (walk_smem > 48 * 1024) cudaFuncSetAttribute(k_delta_walk<RS_, PLAIN_, HEADG_>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)walk_smem); \
+        launch_pdl(k_delta_walk<RS_, PLAIN_, HEADG_>, dim3((vdim + wcols - 1) / wcols, H), dim3(kWalkThreads), walk_smem, st, dst, bufs[s.buf[1]], \
+                   scratch, bufs[s.buf[6]], bufs[s.buf[7]], T, H, dim, vdim, s.off[2], s.n[5], dst_rs);                                         \
+    } while (0)
 #define ZG_WALK(RS_)                                                                                                                            \
     case RS_:                                                                                                                                   \
-        if (form & kDeltaPlain) {                                                                                                               \
-            if (walk_smem > 48 * 1024) cudaFuncSetAttribute(k_delta_walk<RS_, true>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)walk_smem); \
-            launch_pdl(k_delta_walk<RS_, true>, dim3((vdim + wcols - 1) / wcols, H), dim3(kWalkThreads), walk_smem, st, dst, bufs[s.buf[1]],    \
-                       scratch, bufs[s.buf[6]], bufs[s.buf[7]], T, H, dim, vdim, s.off[2], s.n[5], dst_rs);                                     \
-        } else {                                                                                                                                \
-            if (walk_smem > 48 * 1024) cudaFuncSetAttribute(k_delta_walk<RS_, false>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)walk_smem); \
-            launch_pdl(k_delta_walk<RS_, false>, dim3((vdim + wcols - 1) / wcols, H), dim3(kWalkThreads), walk_smem, st, dst, bufs[s.buf[1]],   \
-                       scratch, bufs[s.buf[6]], bufs[s.buf[7]], T, H, dim, vdim, s.off[2], s.n[5], dst_rs);                                     \
-        }                                                                                                                                       \
+        if (form & kDeltaPlain) { if (form & kDeltaHeadDecay) ZG_WALK_FORM(RS_, true, true); else ZG_WALK_FORM(RS_, true, false); }             \
+        else if (form & kDeltaHeadDecay) ZG_WALK_FORM(RS_, false, true);                                                                        \
+        else ZG_WALK_FORM(RS_, false, false);                                                                                                   \
         break;
                 switch (WS) { ZG_WALK(1) ZG_WALK(2) ZG_WALK(4) ZG_WALK(8) ZG_WALK(16) default: ZG_WALK(32) }
 #undef ZG_WALK
+#undef ZG_WALK_FORM
             } else ZG_SEQ_WDT(s.n[9], {
                 if (smem > 48 * 1024) cudaFuncSetAttribute(k_delta_rule<WT>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
-                launch_pdl(k_delta_rule<WT>, dim3(grid), dim3(kDeltaThreads), smem, st, dst, bufs[s.buf[1]], betab, bufs[s.buf[3]], wptr<WT>(bufs, s.buf[5], 0), bufs[s.buf[6]],
+                launch_pdl(k_delta_rule<WT>, dim3(grid), dim3(kDeltaThreads), smem, st, dst, bufs[s.buf[1]], betab, bufs[s.buf[3]] + s.n[13], wptr<WT>(bufs, s.buf[5], 0), bufs[s.buf[6]],
                                                                   bufs[s.buf[7]], T, H, G, dim, vdim, RS, s.off[0], s.off[1], s.off[2], s.off[3], s.off[4], s.off[5],
                                                                   s.n[5], s.n[6], s.n[7], s.f[1], s.f[2], form, inv_tau, dst_rs);
             });

@@ -51,6 +51,14 @@ def _open_pepevik(be, path, dtype, n_slots, max_chunk, max_tokens):
     return SequenceSession(be, model, n_slots=n_slots, max_chunk=max_chunk, max_context=max_tokens or None)
 
 
+@register("Fotovik")
+def _open_fotovik(be, path, dtype, n_slots, max_chunk, max_tokens):
+    from .fotovik import FotovikModel
+    from .session import SequenceSession
+    model = FotovikModel.load(be, path, dtype)
+    return SequenceSession(be, model, n_slots=n_slots, max_chunk=max_chunk, max_context=max_tokens or None)
+
+
 @register("Setirax")
 def _open_setirax(be, path, dtype, n_slots, max_chunk, max_tokens):
     from .session import SequenceSession

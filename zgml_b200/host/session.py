@@ -10,7 +10,7 @@ A model object provides
 
 `SequenceSession.feed(request, tokens, want)` cuts the request's next tokens into chunks from a fixed menu of program
 sizes (powers of two up to `max_chunk`, compiled on first use and kept), writes the control buffer (position, state slot,
-token ids) and executes; the CUDA graph of a program is replayed unchanged from step to step.  How a prompt is cut
+previous token, token ids) and executes; the CUDA graph of a program is replayed unchanged from step to step.  How a prompt is cut
 changes nothing but rounding: state is carried exactly, and every chunk attends through the same key ring.
 `step(entries, end)` is the batch form (requests are advanced one after the other, each alone in its program, so a
 request's logits cannot depend on its neighbours); `generate` is greedy / sampled decoding on top of `feed`.
@@ -79,9 +79,9 @@ class SequenceSession:
             self._programs[key] = (lp, handle, ctl, logits)
         return self._programs[key]
 
-    def _run(self, T, head, slot, pos, tokens):
+    def _run(self, T, head, slot, pos, prev, tokens):
         lp, handle, ctl, logits = self.program(T, head)
-        ctl[abi.CTL_POS], ctl[abi.CTL_SLOT] = pos, slot
+        ctl[abi.CTL_POS], ctl[abi.CTL_SLOT], ctl[abi.CTL_PREV] = pos, slot, prev
         ctl[abi.CTL_IDS:] = tokens
         outs = [ProgramIO(lp.buf_logits, logits)] if logits is not None else []
         self.be.execute_program(handle, [ProgramIO(lp.buf_ctl, ctl)], outs)
@@ -106,10 +106,10 @@ class SequenceSession:
         for T in cut(len(tokens), self.menu):
             local = sorted({w - at for w in want if at <= w < at + T})
             head = "none" if not local else ("last" if local == [T - 1] else "all")
-            logits = self._run(T, head, slot, self.pool.position(request_id), tokens[at:at + T])
+            logits = self._run(T, head, slot, self.pool.position(request_id), self.pool.last_token(request_id), tokens[at:at + T])
             for w in local:
                 rows[at + w] = logits[0 if head == "last" else w].copy()
-            self.pool.advance(request_id, T)
+            self.pool.advance(request_id, T, tokens[at + T - 1])
             at += T
         return np.stack([rows[w] for w in want]) if want else np.zeros((0, self.model.vocab), np.float32)
 

@@ -32,7 +32,6 @@ rglru       [y | x] = W h + b in ONE matmul; CAUSAL_CONV (bias) over x; the two 
             over the stacked blocks; RG_LRU (tanh-GELU of y on the way out); W_o.
 """
 import json
-import math
 import os
 from dataclasses import dataclass
 from typing import Dict, List, Optional
@@ -41,6 +40,7 @@ import numpy as np
 
 from .. import abi
 from ..backend import CudaBackend, DeviceBuffer, DeviceOp, DeviceProgram, ExternBuffer
+from .rotary import rotary_frequencies
 from .safetensors import SafetensorsFile
 from .session import LoweredProgram
 from .state import SequenceStatePool, StateSpec
@@ -51,22 +51,6 @@ DEFAULT_CONTEXT = 4096     # positions a sequence may reach when a layer attends
 MIXERS = ("latent_attention", "parallel", "rglru")
 LRU_RATE = 8.0             # log a = -8 r softplus(lam): fixed by the design
 EXPAND_MIN_TOKENS = 128    # steps from this size on expand a latent layer's keys and values per head (bfloat16 sessions)
-
-
-def rotary_frequencies(rot: dict) -> np.ndarray:
-    """[dims / 2] f32: pair i turns by p * f_i, f_i = base^(-2i / dims).  With `scaling` (factor, low, high, original): a pair whose
-    wavelength 2 pi / f is shorter than original / high keeps f, one longer than original / low turns `factor` times slower, and
-    in between the two are blended linearly in original / wavelength."""
-    dims = int(rot["dims"])
-    f = float(rot["base"]) ** (-2.0 * np.arange(dims // 2, dtype=np.float64) / dims)
-    sc = rot.get("scaling")
-    if sc:
-        factor, low, high, original = float(sc["factor"]), float(sc["low"]), float(sc["high"]), float(sc["original"])
-        wl = 2.0 * math.pi / f
-        blend = (original / wl - low) / (high - low) if high != low else np.ones_like(f)
-        mixed = (1.0 - blend) * f / factor + blend * f
-        f = np.where(wl < original / high, f, np.where(wl > original / low, f / factor, mixed))
-    return f.astype(np.float32)
 
 
 def _tensor_sizes(kind: str, m: dict, mlp: Optional[dict]) -> tuple:
