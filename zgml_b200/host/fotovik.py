@@ -414,3 +414,81 @@ class FotovikModel:
         for b in list(self.buffers.values()) + list(self._freqs.values()) + list(self._decays.values()):
             b.free()
         self.buffers, self._freqs, self._decays = {}, {}, {}
+
+
+def synthetic_config(width: int, n_layers: int, heads: int, kv_heads: int, dim: int, ff: int, vocab: int, window: int = 1024, pool: int = 32,
+                     lightning_heads: Optional[int] = None, delta_heads: Optional[int] = None, conv: int = 4, loop: Optional[dict] = None) -> dict:
+    """config.json contents of a random-init model: layers cycle the pair, window attention and the delta rule; every layer has a
+    dense feed-forward."""
+    layers = []
+    for i in range(n_layers):
+        kind = ("parallel", "attention", "delta")[i % 3]
+        if kind == "parallel":
+            left = {"dim": dim, "heads": heads, "kv_heads": kv_heads, "rot": {"base": 10000.0, "dims": dim // 2, "scaling": {"factor": 2.0}}, "scale": dim ** -0.5, "vdim": dim}
+            n = lightning_heads or max(1, heads // 2)
+            mixer = {"left": left, "right": {"decay": [1.0 - 2.0 ** -(3.0 + 5.0 * h / n) for h in range(n)], "dim": dim, "heads": n, "vdim": dim}}
+        elif kind == "attention":
+            mixer = {"dim": dim, "heads": heads, "kv_heads": kv_heads, "mask": {"pool": pool, "size": window}, "rot": {"base": 10000.0, "dims": dim}, "scale": dim ** -0.5, "vdim": dim}
+        else:
+            n = delta_heads or heads
+            mixer = {"conv": conv, "dim": dim, "heads": n, "kv_heads": max(1, n // 2), "vdim": dim}
+        layers.append({"type": kind, "mixer": mixer, "mlp": {"kind": "dense", "ff": ff}})
+    return {"architecture": ARCHITECTURE, "vocab": vocab, "width": width, "norm": {"eps": 1e-5}, "layers": layers, "loop": loop,
+            "embedding": {"scale": 1.0, "bigram": {"buckets": 4093, "mul_prev": 1009, "mul_cur": 31}}}
+
+
+def synthetic_tensors(cfg: dict, seed: int = 0):
+    """Accessor name -> random f32 tensor of the shape the configuration implies (benchmarks and smoke runs; values are scaled like a
+    trained model's so that activations stay O(1))."""
+    import zlib
+    D = cfg["width"]
+
+    def attention_shapes(m):
+        H, G, d, dv = m["heads"], m["kv_heads"], m["dim"], m["vdim"]
+        return {"q": (H * d, D), "k": (G * d, D), "v": (G * dv, D), "q.norm": (d,), "k.norm": (d,), "sink": (H,), "o": (D, H * dv)}
+
+    def shape_of(name):
+        top = {"embed": (cfg["vocab"], D), "head": (cfg["vocab"], D), "final.norm": (), "bigram": (cfg["embedding"]["bigram"]["buckets"] + 1, D)}
+        if name in top:
+            return top[name]
+        layer, rest = name.split(".", 1)
+        L = cfg["layers"][int(layer[1:])]
+        m = L["mixer"]
+        if rest.startswith("norm"):
+            return ()
+        if rest.startswith("mlp."):
+            return {"up": (L["mlp"]["ff"], D), "down": (D, L["mlp"]["ff"])}[rest[4:]]
+        t = rest[len("mix."):]
+        if L["type"] == "attention":
+            return attention_shapes(m)[t]
+        if L["type"] == "delta":
+            H, G, d, dv, taps = m["heads"], m["kv_heads"], m["dim"], m["vdim"], m["conv"]
+            return {"q": (G * d, D), "k": (G * d, D), "v": (H * dv, D), "q.conv": (G * d, taps), "k.conv": (G * d, taps), "v.conv": (H * dv, taps), "b": (H, D), "a": (H, D), "A_log": (H,),
+                    "dt_bias": (H,), "norm": (dv,), "g": (H * dv, D), "o": (D, H * dv)}[t]
+        if t.endswith(".out"):
+            return (D,)
+        if t.startswith("left."):
+            return attention_shapes(m["left"])[t[5:]]
+        H, d, dv = m["right"]["heads"], m["right"]["dim"], m["right"]["vdim"]
+        return {"q": (H * d, D), "k": (H * d, D), "v": (H * dv, D), "g": (H * dv, D), "norm": (H * dv,), "o": (D, H * dv)}[t[6:]]
+
+    def get(name):
+        shp = shape_of(name)
+        r = np.random.default_rng([seed, zlib.crc32(name.encode())])
+        last = name.rsplit(".", 1)[-1]
+        if last.startswith("norm") or last == "out":
+            return np.ones(shp, np.float32)
+        if last == "conv":
+            a = (r.random(shp, dtype=np.float32) - 0.5) * 0.5
+            a[:, -1] += 1.0
+            return a
+        if last in ("A_log", "dt_bias"):
+            return (-3.0 + 2.0 * r.random(shp, dtype=np.float32)).astype(np.float32)
+        if last == "sink":
+            return (r.random(shp, dtype=np.float32) * 0.2).astype(np.float32)
+        a = r.random(shp, dtype=np.float32)
+        a -= 0.5
+        a *= np.float32(np.sqrt(12.0 / (1 if name in ("embed", "bigram") else shp[-1])))
+        return a
+
+    return get
