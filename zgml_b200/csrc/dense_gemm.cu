@@ -86,17 +86,25 @@ __global__ void k_to_bf16(const float* __restrict__ x, uint32_t x_rs, uint32_t* 
     }
 }
 
-// the epilogue's activation (the kinds of the ACTIVATION op, shifted by one: 0 is none)
-__device__ __forceinline__ float gemm_act(float z, uint32_t act, float p) {
-    switch (act) {
-        case 5: return p * tanhf(z / p);
-        case 0: return z;
-        case 1: { const float r = fmaxf(z, 0.0f); return r * r; }
-        case 2: return z / (1.0f + expf(-z));
-        case 3: return 0.5f * z * (1.0f + tanhf(0.7978845608028654f * fmaf(0.044715f * z * z, z, z)));
-        case 6: return 0.5f * z * (1.0f + erff(z * 0.7071067811865476f));
-        default: return fmaxf(z, 0.0f);
+// the epilogue's activation (the kinds of the ACTIVATION op, shifted by one: 0 is none), a compile-time kind: 128 outputs per
+// epilogue thread pass it one after the other, so what counts is straight-line code whose chains interleave.  (A switch inside the
+// loop cost 340 cycles per output.)  Exponentials and quotients are the fast intrinsics: the product's inputs are bfloat16.
+// The exact GELU takes erf from Abramowitz and Stegun, Handbook of Mathematical Functions, formula 7.1.26 (absolute error below
+// 1.5e-7): 1 - erf(x) = (a1 t + ... + a5 t^5) exp(-x^2), t = 1 / (1 + p x), x >= 0.
+template <int ACT>
+__device__ __forceinline__ float gemm_act(float z, float p) {
+    if (ACT == 1) { const float r = fmaxf(z, 0.0f); return r * r; }
+    if (ACT == 2) return __fdividef(z, 1.0f + __expf(-z));
+    if (ACT == 3) return 0.5f * z * (1.0f + tanhf(0.7978845608028654f * fmaf(0.044715f * z * z, z, z)));
+    if (ACT == 4) return fmaxf(z, 0.0f);
+    if (ACT == 5) return p * tanhf(z / p);
+    if (ACT == 6) {
+        const float x = fabsf(z) * 0.7071067811865476f, t = __fdividef(1.0f, fmaf(0.3275911f, x, 1.0f));
+        const float poly = t * fmaf(t, fmaf(t, fmaf(t, fmaf(t, 1.061405429f, -1.453152027f), 1.421413741f), -0.284496736f), 0.254829592f);
+        const float tail = poly * __expf(-x * x);      // 1 - erf(x)
+        return 0.5f * z * (z < 0.0f ? tail : 2.0f - tail);
     }
+    return z;
 }
 struct GemmParams {
     float* out;
@@ -110,7 +118,7 @@ struct GemmParams {
 
 // GROUPED: the rows are sorted by weight matrix (expert) in whole 128-row tiles; tile t multiplies with matrix tile_group[t]
 // of the stacked [groups][N][K] weight tensor.
-template <bool GROUPED, bool ACT>       // ACT: the epilogue applies p.act (its own instantiation: the plain epilogue stays as it was)
+template <bool GROUPED, int ACT>        // ACT: the activation of the epilogue (GemmParams::act; one instantiation each)
 __global__ void __launch_bounds__(kThreads, 1)
 dense_gemm_kernel(const __grid_constant__ CUtensorMap tmap_a, const __grid_constant__ CUtensorMap tmap_b, const GemmParams p) {
     int group = 0;
@@ -182,7 +190,6 @@ dense_gemm_kernel(const __grid_constant__ CUtensorMap tmap_a, const __grid_const
         const bool ok = mbar_wait(tmem_full, 0);
         asm volatile("tcgen05.fence::after_thread_sync;" ::: "memory");
         const uint32_t m_base = tile_m * BM + quarter * 32;
-        auto finish = [&](float z, uint32_t n) { return ACT && n >= p.act_lo && n < p.act_hi ? gemm_act(z, p.act, p.act_p) : z; };
         uint4* tb = reinterpret_cast<uint4*>(dsm_raw + (base - smem_u32(dsm_raw)) + ew * (32 * 36 * 4));   // the stages are idle now
 #pragma unroll 1
         for (uint32_t c0 = 0; ok && c0 < BN; c0 += 32) {
@@ -202,11 +209,18 @@ dense_gemm_kernel(const __grid_constant__ CUtensorMap tmap_a, const __grid_const
             for (int i = 0; i < 8; i++) tb[lane * 9 + i] = make_uint4(v[4 * i], v[4 * i + 1], v[4 * i + 2], v[4 * i + 3]);
             __syncwarp();
             const uint32_t n0 = tile_n * BN + c0;
+            const bool some = ACT && n0 < p.act_hi && n0 + 32 > p.act_lo;     // uniform: whether any of these columns takes the activation
+            auto finish = [&](float z, uint32_t n) {
+                if (!ACT) return z;
+                const float a = gemm_act<ACT>(z, p.act_p);
+                return n >= p.act_lo && n < p.act_hi ? a : z;
+            };
             if (n0 < p.N) {
                 if (p.out_vec4 && n0 + 32 <= p.N) {
                     const uint32_t nn = n0 + 4 * (lane & 7);
                     float b[4] = {0.0f, 0.0f, 0.0f, 0.0f};
                     if (p.bias) for (int j = 0; j < 4; j++) b[j] = __bfloat162float(p.bias[nn + j]);
+                    if (!ACT || some) {
 #pragma unroll
                     for (int it = 0; it < 8; it++) {
                         const uint32_t rr = it * 4 + (lane >> 3), mm = m_base + rr;
@@ -214,6 +228,15 @@ dense_gemm_kernel(const __grid_constant__ CUtensorMap tmap_a, const __grid_const
                         const float4 f = make_float4(finish(__uint_as_float(o.x) + b[0], nn), finish(__uint_as_float(o.y) + b[1], nn + 1), finish(__uint_as_float(o.z) + b[2], nn + 2),
                                                      finish(__uint_as_float(o.w) + b[3], nn + 3));
                         if (mm < p.M) *reinterpret_cast<float4*>(p.out + (size_t)mm * p.out_rs + nn) = f;
+                    }
+                    } else {
+#pragma unroll
+                    for (int it = 0; it < 8; it++) {
+                        const uint32_t rr = it * 4 + (lane >> 3), mm = m_base + rr;
+                        const uint4 o = tb[rr * 9 + (lane & 7)];
+                        const float4 f = make_float4(__uint_as_float(o.x) + b[0], __uint_as_float(o.y) + b[1], __uint_as_float(o.z) + b[2], __uint_as_float(o.w) + b[3]);
+                        if (mm < p.M) *reinterpret_cast<float4*>(p.out + (size_t)mm * p.out_rs + nn) = f;
+                    }
                     }
                 } else if (n0 + lane < p.N) {
                     const uint32_t* tw = reinterpret_cast<const uint32_t*>(tb);
@@ -235,6 +258,10 @@ typedef CUresult (*EncodeTiledFn)(CUtensorMap*, CUtensorMapDataType, cuuint32_t,
                                   CUtensorMapL2promotion, CUtensorMapFloatOOBfill);
 EncodeTiledFn g_encode = nullptr;
 bool g_attr_set = false;
+constexpr int kActs = 7;
+typedef void (*GemmKernel)(const CUtensorMap, const CUtensorMap, const GemmParams);
+const GemmKernel g_kernel[kActs] = {dense_gemm_kernel<false, 0>, dense_gemm_kernel<false, 1>, dense_gemm_kernel<false, 2>, dense_gemm_kernel<false, 3>,
+                                    dense_gemm_kernel<false, 4>, dense_gemm_kernel<false, 5>, dense_gemm_kernel<false, 6>};   // by activation
 
 bool prepare() {
     if (!g_encode) {
@@ -247,9 +274,8 @@ bool prepare() {
         g_encode = (EncodeTiledFn)fn;
     }
     if (!g_attr_set) {
-        cudaError_t e = cudaFuncSetAttribute(dense_gemm_kernel<false, false>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)kSmem);
-        if (e == cudaSuccess) e = cudaFuncSetAttribute(dense_gemm_kernel<false, true>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)kSmem);
-        if (e == cudaSuccess) e = cudaFuncSetAttribute(dense_gemm_kernel<true, false>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)kSmem);
+        cudaError_t e = cudaFuncSetAttribute(dense_gemm_kernel<true, 0>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)kSmem);
+        for (int k = 0; k < kActs && e == cudaSuccess; k++) e = cudaFuncSetAttribute(g_kernel[k], cudaFuncAttributeMaxDynamicSharedMemorySize, (int)kSmem);
         if (e != cudaSuccess) { zg_set_error("cudaFuncSetAttribute(dense_gemm) failed: %s", cudaGetErrorString(e)); return false; }
         g_attr_set = true;
     }
@@ -302,8 +328,8 @@ bool zg_dense_gemm_launch(const void* w_bf16, const void* bias_bf16, const float
     p.out_vec4 = ((reinterpret_cast<uintptr_t>(dst) & 15) == 0 && (dst_rs & 3) == 0) ? 1u : 0u;
     p.tile_group = nullptr;
     dim3 grid((N + BN - 1) / BN, (M + BM - 1) / BM);
-    if (act) dense_gemm_kernel<false, true><<<grid, kThreads, kSmem, st>>>(map_a, map_b, p);
-    else dense_gemm_kernel<false, false><<<grid, kThreads, kSmem, st>>>(map_a, map_b, p);
+    if (act >= (uint32_t)kActs) { zg_set_error("dense gemm: unknown activation %u", act); return false; }
+    g_kernel[act]<<<grid, kThreads, kSmem, st>>>(map_a, map_b, p);
     ZG_COUNT_LAUNCH();
     cudaError_t e = cudaGetLastError();
     if (e != cudaSuccess) { zg_set_error("dense gemm launch failed: %s", cudaGetErrorString(e)); return false; }
@@ -337,7 +363,7 @@ bool zg_dense_gemm_grouped_launch(const void* w_bf16, uint32_t groups, const voi
     p.out_vec4 = ((reinterpret_cast<uintptr_t>(dst) & 15) == 0 && (dst_rs & 3) == 0) ? 1u : 0u;
     p.tile_group = d_tile_group;
     dim3 grid((N + BN - 1) / BN, rows / BM);
-    dense_gemm_kernel<true, false><<<grid, kThreads, kSmem, st>>>(map_a, map_b, p);
+    dense_gemm_kernel<true, 0><<<grid, kThreads, kSmem, st>>>(map_a, map_b, p);
     ZG_COUNT_LAUNCH();
     cudaError_t e = cudaGetLastError();
     if (e != cudaSuccess) { zg_set_error("grouped dense gemm launch failed: %s", cudaGetErrorString(e)); return false; }

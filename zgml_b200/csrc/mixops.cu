@@ -77,7 +77,7 @@ __device__ void pool_block(float* __restrict__ pooled, const float* __restrict__
     float* out = pooled + ((size_t)slot * pool_rows + end - 1) * width;
     for (uint32_t c = first; c < cols; c += stride) {
         float sum = 0.0f;
-#pragma unroll 4
+#pragma unroll 16
         for (uint32_t r = 0; r < P; r++) sum += rows[(size_t)(((end - 1) * P + r) % R) * width + c];
         out[c] = sum / (float)P;
     }
@@ -95,8 +95,8 @@ __global__ void k_cache_append(float* __restrict__ cache, const float* __restric
                                float base, uint32_t norm_group, float* qsrc, const WT* __restrict__ qw, uint32_t q_heads, uint32_t temp_every, float temp_coef,
                                uint32_t hrot, const float* __restrict__ freqs, uint32_t horder, float* __restrict__ pooled, uint32_t pool, uint32_t pool_rows) {
     pdl_enter();
-    if (pooled && blockIdx.x == gridDim.x - 1) {       // single-token steps: one more CTA averages the block that ended just before this token
-        pool_block(pooled, cache, ctl, 1u, cols, width, R, pool, pool_rows, 0u, threadIdx.x, blockDim.x);
+    if (pooled && blockIdx.x) {       // single-token steps: further CTAs average the block that ended just before this token
+        pool_block(pooled, cache, ctl, 1u, cols, width, R, pool, pool_rows, 0u, (blockIdx.x - 1) * blockDim.x + threadIdx.x, (gridDim.x - 1) * blockDim.x);
         return;
     }
     __shared__ float sh[32];
@@ -529,10 +529,12 @@ __global__ void __launch_bounds__(kCtThreads) k_cached_attention_tiled(CaArgs a,
 // merge of the key shares: CTA (x, y) = 128 value columns y of (token, head, map) x; a share that saw no key carries
 // max = -inf and weighs nothing (its output is zero)
 // (a: for the sink, the output scale and the row layout of dst; HM = H * maps)
-__global__ void __launch_bounds__(128) k_cached_attention_merge(CaArgs a, const float* __restrict__ part, uint32_t dv, uint32_t splits,
+constexpr int kMergeGroups = 4;        // groups of 128 threads that each add up a quarter of the shares
+__global__ void __launch_bounds__(128 * kMergeGroups) k_cached_attention_merge(CaArgs a, const float* __restrict__ part, uint32_t dv, uint32_t splits,
                                                                 uint32_t wkind) {
     pdl_enter();
-    __shared__ float w[kCtMaxSplits];
+    __shared__ float w[kCtMaxSplits], sums[kMergeGroups][128];
+    const uint32_t group = threadIdx.x >> 7, c = blockIdx.y * 128 + (threadIdx.x & 127);
     const float* P = part + (size_t)blockIdx.x * splits * (4 + dv);
     const uint32_t HM = a.H * a.maps, hm = blockIdx.x % HM;
     if (wkind) {                                       // unnormalised weights: the shares just add up
@@ -547,11 +549,16 @@ __global__ void __launch_bounds__(128) k_cached_attention_merge(CaArgs a, const 
         if (threadIdx.x + 32 < splits) w[threadIdx.x + 32] = e1 * inv;
     }
     __syncthreads();
-    const uint32_t c = blockIdx.y * 128 + threadIdx.x;
-    if (c >= dv) return;
     float acc = 0.0f;
-#pragma unroll 4
-    for (uint32_t i = 0; i < splits; i++) acc = fmaf(P[i * (4 + dv) + 4 + c], w[i], acc);
+    if (c < dv) {
+#pragma unroll 16
+        for (uint32_t i = group; i < splits; i += kMergeGroups) acc = fmaf(P[i * (4 + dv) + 4 + c], w[i], acc);
+    }
+    sums[group][threadIdx.x & 127] = acc;
+    __syncthreads();
+    if (group || c >= dv) return;
+#pragma unroll
+    for (int g = 1; g < kMergeGroups; g++) acc += sums[g][threadIdx.x];
     a.dst[(size_t)(blockIdx.x / HM) * a.dst_rs + (size_t)hm * dv + c] = acc;
 }
 
@@ -1061,7 +1068,7 @@ bool zg_launch_mix_op(const ZgOp& op, float* const* bufs, float* scratch, cudaSt
         case ZG_OP_CACHE_APPEND: {
             float* pooled = s.n[11] ? bufs[s.buf[5]] + s.off[1] : nullptr;
             const bool turn_only = s.n[13] == 2;
-            ZG_SEQ_WDT(s.n[5] ? s.n[7] : ZG_W_F32, launch_pdl(k_cache_append<WT>, dim3(s.n[0] + (pooled && s.n[0] == 1 ? 1 : 0)), dim3(s.off[5] ? 256 : 128), (size_t)s.n[10] * sizeof(float), st, bufs[s.buf[0]] + s.off[1], bufs[s.buf[1]] + s.off[0], bufs[s.buf[2]],
+            ZG_SEQ_WDT(s.n[5] ? s.n[7] : ZG_W_F32, launch_pdl(k_cache_append<WT>, dim3(s.n[0] + (pooled && s.n[0] == 1 ? (s.n[1] + 255) / 256 : 0)), dim3(s.off[5] ? 256 : 128), (size_t)s.n[10] * sizeof(float), st, bufs[s.buf[0]] + s.off[1], bufs[s.buf[1]] + s.off[0], bufs[s.buf[2]],
                                                              s.n[5] && !turn_only ? wptr<WT>(bufs, s.buf[3], s.off[2]) : nullptr, s.n[1], s.n[2], s.n[3], s.n[4], s.n[5], s.n[6], s.n[8], s.f[0], s.f[1], s.n[9],
                                                              s.off[5] ? bufs[s.buf[1]] + s.off[3] : nullptr, s.off[5] && !turn_only ? wptr<WT>(bufs, s.buf[3], s.off[4]) : nullptr, s.off[5], s.off[6], s.f[2],
                                                              s.n[10], s.n[10] && s.buf[4] != ZG_NO_BUF ? (const float*)(bufs[s.buf[4]] + s.off[7]) : (const float*)nullptr, s.n[13],
@@ -1102,7 +1109,7 @@ bool zg_launch_mix_op(const ZgOp& op, float* const* bufs, float* scratch, cudaSt
 #undef ZG_CF
                 if (S > 1) {
                     ZG_SEQ_CHECK();
-                    launch_pdl(k_cached_attention_merge, dim3(a.T * a.H * a.maps, (a.dv + 127) / 128), dim3(128), 0, st, a, (const float*)part, a.dv, S, a.wkind);
+                    launch_pdl(k_cached_attention_merge, dim3(a.T * a.H * a.maps, (a.dv + 127) / 128), dim3(128 * kMergeGroups), 0, st, a, (const float*)part, a.dv, S, a.wkind);
                 }
             } else if (aligned) {
                 const uint32_t S = scratch ? ca_splits(s) : 1;
@@ -1123,7 +1130,7 @@ bool zg_launch_mix_op(const ZgOp& op, float* const* bufs, float* scratch, cudaSt
                 }
                 if (S > 1) {
                     ZG_SEQ_CHECK();
-                    launch_pdl(k_cached_attention_merge, dim3(a.T * a.H * a.maps, (a.dv + 127) / 128), dim3(128), 0, st, a, (const float*)part, a.dv, S, a.wkind);
+                    launch_pdl(k_cached_attention_merge, dim3(a.T * a.H * a.maps, (a.dv + 127) / 128), dim3(128 * kMergeGroups), 0, st, a, (const float*)part, a.dv, S, a.wkind);
                 }
             } else {
                 const uint32_t warps = 4, items = a.T * a.H * a.maps;

@@ -34,6 +34,18 @@ __device__ float block_sum(float v, float* sh) {
     for (int i = 0; i < nw; i++) r += sh[i];
     return r;
 }
+// two sums at once
+__device__ __forceinline__ float2 block_sum2(float a, float b, float* sh) {
+    const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5, nw = (blockDim.x + 31) >> 5;   // at most 16 warps: sh holds 32 floats
+    a = warp_sum(a);
+    b = warp_sum(b);
+    __syncthreads();
+    if (lane == 0) { sh[2 * warp] = a; sh[2 * warp + 1] = b; }
+    __syncthreads();
+    float2 r = make_float2(0.0f, 0.0f);
+    for (int i = 0; i < nw; i++) { r.x += sh[2 * i]; r.y += sh[2 * i + 1]; }
+    return r;
+}
 // Programmatic dependent launch (as the framework's other program kernels do): let the next kernel of the stream become
 // resident while this one runs, and hold this one until its predecessor has completed.  Nothing is read before the wait.
 __device__ __forceinline__ void pdl_enter() {

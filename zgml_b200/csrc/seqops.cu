@@ -17,24 +17,18 @@ template <typename WT>
 __global__ void k_embed(float* __restrict__ dst, const float* __restrict__ ctl, const WT* __restrict__ table, uint32_t D, float scale,
                         const WT* __restrict__ positions, const WT* __restrict__ bigram, uint32_t buckets, uint32_t mul_prev, uint32_t mul_cur) {
     pdl_enter();
-    const uint32_t t = blockIdx.x;
-    const size_t row = (size_t)ctl_word(ctl, ZG_CTL_IDS + t) * D;
+    const uint32_t t = blockIdx.x, c = blockIdx.y * blockDim.x + threadIdx.x;
+    if (c >= D) return;
+    const int id = ctl_word(ctl, ZG_CTL_IDS + t);
+    float add = 0.0f;
     if (bigram) {          // a row chosen by a hash of the previous and the current token, not scaled; a sequence's first token takes the last row
         const int prev = t ? ctl_word(ctl, ZG_CTL_IDS + t - 1) : ctl_word(ctl, ZG_CTL_PREV);
-        const unsigned long long cur = (unsigned long long)ctl_word(ctl, ZG_CTL_IDS + t);
-        const unsigned long long b = prev < 0 ? (unsigned long long)buckets : ((unsigned long long)prev * mul_prev + cur * mul_cur) % buckets;
-        const size_t brow = (size_t)b * D;
-#pragma unroll 4
-        for (uint32_t c = threadIdx.x; c < D; c += blockDim.x) dst[(size_t)t * D + c] = fmaf(wld(table, row + c), scale, wld(bigram, brow + c));
-        return;
+        const unsigned long long b = prev < 0 ? (unsigned long long)buckets : ((unsigned long long)prev * mul_prev + (unsigned long long)id * mul_cur) % buckets;
+        add = wld(bigram, (size_t)b * D + c);
+    } else if (positions) {       // a learned position row, not scaled
+        add = wld(positions, ((size_t)ctl_word(ctl, ZG_CTL_POS) + t) * D + c);
     }
-    if (positions) {       // a learned position row, not scaled
-        const size_t prow = ((size_t)ctl_word(ctl, ZG_CTL_POS) + t) * D;
-#pragma unroll 4
-        for (uint32_t c = threadIdx.x; c < D; c += blockDim.x) dst[(size_t)t * D + c] = fmaf(wld(table, row + c), scale, wld(positions, prow + c));
-        return;
-    }
-    for (uint32_t c = threadIdx.x; c < D; c += blockDim.x) dst[(size_t)t * D + c] = wld(table, row + c) * scale;
+    dst[(size_t)t * D + c] = fmaf(wld(table, (size_t)id * D + c), scale, add);
 }
 
 // ── LINEAR, few rows (decode): one warp per output feature, the weight row streamed once for all rows ─────────────────
@@ -378,6 +372,21 @@ __global__ void __launch_bounds__(256) k_norm_any_rows(float* dst, const float* 
         norm_any_pass(dst2 + row, dst + row, (const float*)nullptr, w2, cols, kind2, eps, gain, sh, (const float*)nullptr, (const WT*)nullptr);
     }
 }
+// A thread's share of a weight, or of one value for all columns (kind bit 5).  The column is clamped instead of tested and whether the
+// weight is there at all is decided once, so that all loads are in flight before the first is widened; shares past the row are unused.
+template <typename WT, int kKeep>
+__device__ __forceinline__ void norm_any_weights(float (&out)[kKeep], const WT* __restrict__ w, bool have, uint32_t cols, uint32_t kind) {
+    if (!have) {
+#pragma unroll
+        for (int i = 0; i < kKeep; i++) out[i] = 0.0f;
+        return;
+    }
+    WT raw[kKeep];
+#pragma unroll
+    for (int i = 0; i < kKeep; i++) raw[i] = w[norm_col(min(threadIdx.x + i * blockDim.x, cols - 1), kind)];
+#pragma unroll
+    for (int i = 0; i < kKeep; i++) out[i] = wld(raw + i, 0);
+}
 template <typename WT, int kKeep, int kThreads>          // a row of up to kKeep x kThreads values lives in registers (fewer kept values, more CTAs per SM)
 __global__ void __launch_bounds__(kThreads) k_norm_any(float* dst, const float* src, const WT* __restrict__ w, const float* res, uint32_t cols, uint32_t kind, float eps,
                                                   float* dst2, const WT* __restrict__ w2, uint32_t kind2, float gain, const float* src_b, const WT* __restrict__ w_b,
@@ -395,16 +404,11 @@ __global__ void __launch_bounds__(kThreads) k_norm_any(float* dst, const float* 
         return;
     }
     float v[kKeep], wa[kKeep], aux[kKeep], wc[kKeep], bc[kKeep], wo[kKeep];   // aux: the bias of a Dynamic Tanh, or the second source's weight
-#pragma unroll
-    for (int i = 0; i < kKeep; i++) {
-        const uint32_t c = threadIdx.x + i * blockDim.x;
-        const bool in = c < cols;
-        wa[i] = (in && !(kind & 16u)) ? wld(w, norm_col(c, kind)) : 0.0f;
-        aux[i] = in ? ((kind & 8u) ? wld(w, (size_t)cols + c) : (src_b ? wld(w_b, norm_col(c, kind)) : 0.0f)) : 0.0f;
-        wc[i] = (in && dst2 && !(kind2 & 16u)) ? wld(w2, norm_col(c, kind2)) : 0.0f;
-        wo[i] = (in && w_o) ? wld(w_o, norm_col(c, kind_o)) : 0.0f;
-        bc[i] = (in && dst2 && (kind2 & 8u)) ? wld(w2, (size_t)cols + c) : 0.0f;
-    }
+    norm_any_weights<WT, kKeep>(wa, w, !(kind & 16u), cols, kind);
+    norm_any_weights<WT, kKeep>(aux, (kind & 8u) ? w + cols : w_b, (kind & 8u) || src_b, cols, kind);
+    norm_any_weights<WT, kKeep>(wc, w2, dst2 && !(kind2 & 16u), cols, kind2);
+    norm_any_weights<WT, kKeep>(wo, w_o, w_o != nullptr, cols, kind_o);
+    norm_any_weights<WT, kKeep>(bc, w2 + cols, dst2 && (kind2 & 8u), cols, kind2);
     const float alpha = (kind & 8u) ? wld(w, (size_t)2 * cols) : 0.0f, alpha2 = (dst2 && (kind2 & 8u)) ? wld(w2, (size_t)2 * cols) : 0.0f;
     asm volatile("griddepcontrol.wait;" ::: "memory");
     float rv[kKeep], vb[kKeep];
@@ -433,8 +437,17 @@ __global__ void __launch_bounds__(kThreads) k_norm_any(float* dst, const float* 
         inv = 1.0f / sqrtf(block_sum(q, sh) / (float)cols + eps);
     };
     float mean, inv, mean_b = 0.0f, inv_b = 1.0f;
-    stats(v, kind, mean, inv);
-    if (src_b) stats(vb, kind, mean_b, inv_b);
+    if (src_b && (kind & 1u)) {                     // both sources' root mean squares in one reduction
+        float q = 0.0f, qb = 0.0f;
+#pragma unroll
+        for (int i = 0; i < kKeep; i++) { q = fmaf(v[i], v[i], q); qb = fmaf(vb[i], vb[i], qb); }
+        const float2 s2 = block_sum2(q, qb, sh);
+        inv = 1.0f / sqrtf(s2.x / (float)cols + eps); inv_b = 1.0f / sqrtf(s2.y / (float)cols + eps);
+        mean = 0.0f;
+    } else {
+        stats(v, kind, mean, inv);
+        if (src_b) stats(vb, kind, mean_b, inv_b);
+    }
 #pragma unroll
     for (int i = 0; i < kKeep; i++) {
         const uint32_t c = threadIdx.x + i * blockDim.x;
@@ -1614,7 +1627,7 @@ bool zg_launch_seq_op(ZgCudaCtx* ctx, const ZgOp& op, float* const* bufs, float*
     const ZgSeqOp& s = op.u.seq;
     switch (op.tag) {
         case ZG_OP_EMBED:
-            ZG_SEQ_WDT(s.n[2], launch_pdl(k_embed<WT>, dim3(s.n[0]), dim3(128), 0, st, bufs[s.buf[0]], bufs[s.buf[1]], wptr<WT>(bufs, s.buf[2], s.off[0]), s.n[1], s.f[0],
+            ZG_SEQ_WDT(s.n[2], launch_pdl(k_embed<WT>, dim3(s.n[0], (s.n[1] + 255) / 256), dim3(256), 0, st, bufs[s.buf[0]], bufs[s.buf[1]], wptr<WT>(bufs, s.buf[2], s.off[0]), s.n[1], s.f[0],
                                           s.n[3] ? wptr<WT>(bufs, s.buf[2], s.off[1]) : nullptr, s.n[4] ? wptr<WT>(bufs, s.buf[2], s.off[2]) : nullptr, s.n[4], s.n[5], s.n[6]));
             ZG_SEQ_CHECK();
             return true;
