@@ -612,7 +612,7 @@ bool zg_launch_rec_op(const ZgOp& op, float* const* bufs, float* scratch, cudaSt
         }
         case ZG_OP_GATED_NORM: {
             const uint32_t gs = s.n[1] / s.n[2];
-            const uint32_t threads = gs <= 64 ? 32 : (gs <= 512 ? 128 : (gs <= 2048 ? 256 : 512));
+            const uint32_t threads = gs <= 64 ? 32 : (gs <= 1024 ? 128 : (gs <= 2048 ? 256 : 512));   // at most 8 values per thread up to 4096 columns
             ZG_SEQ_WDT(s.n[4], launch_pdl(k_gated_norm<WT>, dim3(s.n[0] * s.n[2]), dim3(threads), 0, st, bufs[s.buf[0]], bufs[s.buf[1]], bufs[s.buf[2]] + s.off[0],
                                           wptr<WT>(bufs, s.buf[3], s.off[1]), s.n[1], s.n[2], s.n[3], s.n[5], s.n[6], s.f[0], s.n[7]));
             ZG_SEQ_CHECK();
