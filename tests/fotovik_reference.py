@@ -135,7 +135,7 @@ def causal_conv(u, w):
 
 
 def delta_rule(q, k, v, beta, g):
-    """q, k [T, H, dim], v [T, H, vdim], beta, g [T, H]: the read-out sees the current token's write."""
+    """q, k [T, H, dim], v [T, H, vdim], beta, g [T, H]: decay, correct towards v, then read."""
     T, H, dim = q.shape
     S = np.zeros((H, dim, v.shape[2]))
     out = np.zeros(v.shape)

@@ -189,7 +189,7 @@ def test_restatement_of_embedding_and_recurrences():
     beta, g = np.array([[0.4], [0.9]]), np.array([[0.5], [0.25]])
     out = ref.delta_rule(q, k, v, beta, g)
     S = np.outer(k[0, 0], 0.4 * v[0, 0])
-    assert np.allclose(out[0, 0], S.T @ q[0, 0])                      # the read-out sees the token's own write
+    assert np.allclose(out[0, 0], S.T @ q[0, 0])                      # read after the token's own write
     S = 0.25 * S
     S = S + np.outer(k[1, 0], 0.9 * (v[1, 0] - S.T @ k[1, 0]))        # corrected after the decay
     assert np.allclose(out[1, 0], S.T @ q[1, 0])
