@@ -86,7 +86,9 @@ typedef enum ZgOpTag {
     ZG_OP_HEAD_NORM = 34,
     ZG_OP_ACTIVATION = 35,
     ZG_OP_RG_LRU = 36,
-    ZG_OP_END = 37
+    /* Stacks with several residual streams (csrc/streamops.cu): the step that closes a sublayer over all of them and opens the next. */
+    ZG_OP_STREAM_STEP = 37,
+    ZG_OP_END = 38
 } ZgOpTag;
 
 /* Parameter pack of the sequence-model ops.  buf[] are program buffer indices (ZG_NO_BUF: absent), off[] element offsets,
@@ -103,15 +105,18 @@ typedef enum ZgOpTag {
  *                   (a second table at off 1 of the same arena, p(t) = the token's position in its sequence)
  *                   with n4 > 0 a row of a bigram table joins it, unscaled: row (previous token * n5 + token * n6) mod n4, and row n4
  *                   (the last of n4 + 1) for a sequence's first token (a third table at off 2; n5, n6 < n4; not together with n3)
- *                   buf 0 dst 1 ctl 2 table | off 0 table 1 positions 2 bigram | n 0 T 1 D 2 wdt 3 positions 4 bigram buckets
- *                   5 factor of the previous token 6 factor of the token | f 0 scale
+ *                   with n7 = 1 the row passes a Dynamic Tanh, tanh(alpha x) * w + b (w, b and alpha in a row at off 3)
+ *                   buf 0 dst 1 ctl 2 table | off 0 table 1 positions 2 bigram 3 norm | n 0 T 1 D 2 wdt 3 positions 4 bigram buckets
+ *                   5 factor of the previous token 6 factor of the token 7 Dynamic Tanh | f 0 scale
  * LINEAR            dst[m, n] = act(sum_k src[m, k] W[n, k] (+ bias[n])); act (n6): 0 none, 1 + the ACTIVATION kind otherwise (f0: its
  *                   parameter, where the kind has one), on the columns [n8, n9) alone (n9 = 0: up to N): a stacked projection whose
  *                   parts differ
  *                   buf 0 dst 1 src 2 W 3 bias 4 ctl | off 0 W 1 bias 2 src 3 dst | n 0 M 1 N 2 K 3 src row stride 4 dst row stride 5 wdt 6 act
- *                   7 source slot stride 8 first column of act 9 end of its columns
+ *                   7 source slot stride 8 first column of act 9 end of its columns 10 pairs 11 row limit
+ *                   With n10 = 1 (gated products) W holds 2 N rows, a gate row and what it multiplies in turns:
+ *                   dst[m, n] = act(sum_k src[m, k] W[2n, k]) * (sum_k src[m, k] W[2n + 1, k]); no bias, no column range.
  *                   With n7 > 0 the source rows are those of a per-sequence state buffer (a ring): n7 elements per slot, the slot
- *                   from the control buffer buf 4.
+ *                   from the control buffer buf 4.  With n11 > 0 rows from position + n11 on are not wanted (and may be left as they are).
  *                   f 0 activation parameter
  * NORM              dst = (res +) norm(src) * w ; kind bit 0 clear: (x - mean) / sqrt(var + eps), set: x / sqrt(mean(x^2) + eps);
  *                   kind bit 1: the weight is stored around zero and applied as (1 + w); kind bit 2: the result is also
@@ -158,14 +163,17 @@ typedef enum ZgOpTag {
  *                   off 0 q 1 k 2 v (columns of a qkv row) 3 beta (column of its row) 4 A_log 5 dt_bias 6 norm_w (weights)
  *                   7 gate (column of its row)
  *                   n 0 T 1 H 2 G 3 dim 4 vdim 5 qkv row stride 6 beta row stride 7 a row stride 8 gate row stride 9 wdt
- *                   10 form 11 dst row stride (0: H * vdim) 12 dst column 13 a (column of its row)
+ *                   10 form 11 dst row stride (0: H * vdim) 12 dst column 13 a (column of its row) 14 bonus (weights)
  *                   f 0 output-norm eps 1 unit-vector eps 2 q scale 3 decay temperature 4 output scale
  *                   Form bits (n10), all clear for the rule above.  Bit 0, plain accumulation (gated linear attention): no
  *                   unit vectors (q is only scaled by f2) and no correction by what the state already holds, u = v:
  *                   S <- g * S + k v^T, o = S^T q; buf 2 is not read.  Bit 1: the decay is g = sigmoid(a + dt_bias)^(1 / f3),
  *                   evaluated as exp(-softplus(-(a + dt_bias)) / f3); A_log is not read.  Bit 2: the output gate is
  *                   silu(gate) instead of sigmoid(gate).  Bit 4: one decay per head instead of one per key channel (a row of buf 3 and
- *                   dt_bias hold H values).  Bit 3: the result is multiplied by f4.  It may land in columns of a
+ *                   dt_bias hold H values).  Bit 5 (with bit 0; RWKV's time mixing): the state is read before the token's write and the token
+ *                   joins through a bonus u per head and key channel: o = S^T q + (sum_i q_i u_i k_i) v, then S <- g * S + k v^T (u: H * dim
+ *                   weights at n14).  Bit 6: the decay is g = exp(-exp(a + dt_bias)); A_log is not read.  Bit 7: norm_w holds H * vdim
+ *                   values, one vector over all heads.  Bit 3: the result is multiplied by f4.  It may land in columns of a
  *                   wider row (n11, n12), beside another mixer's heads.
  * ROUTE             mode 0: s = softmax(logits) over all NE outputs; the `top` largest of s + correction are chosen (ties:
  *                   lowest index); dst[t, c] = {index as int32 bits, s[index]} (weights not renormalised)
@@ -175,8 +183,9 @@ typedef enum ZgOpTag {
  *                   group scores the sum of its two largest choice scores and only outputs of the n7 best groups can be chosen
  *                   (n6 <= 1: no groups); the `top` largest choice scores are chosen (ties: lowest index) and weighted by
  *                   their s divided by (the sum of the chosen s + 1e-20)
+ *                   mode 3: as mode 2, but the chosen s are not divided: each is multiplied by f0
  *                   buf 0 dst [T, top, 2] 1 logits 2 correction | off 0 correction 1 logits | n 0 T 1 NE 2 top 3 logits row
- *                   stride 4 wdt 5 mode 6 groups 7 groups kept
+ *                   stride 4 wdt 5 mode 6 groups 7 groups kept | f 0 factor of the weights (mode 3)
  * MOE_FFN           dst[t] = sum_c weight_c * expert_{index_c}(src[t]); expert e < E: W_down (g * sigmoid(f1 * g) * (u + f2)),
  *                   g = min(W_gate x, f0), u = clamp(W_up x, -f0, f0); index >= E: the identity (x itself).  Expert weights
  *                   are stacked [E, ff, D] (gate, up) and [E, D, ff] (down).
@@ -204,14 +213,17 @@ typedef enum ZgOpTag {
  *                   from the f32 table buf 4 at element off 7, as ROTARY takes it), and the root mean square is that of the
  *                   turned vector: ROTARY fused, for designs that norm after the rotation.  n13 = 1: norm and weight come first and
  *                   the normed vector is turned; n13 = 2: the heads are turned and not normed (no weight is read).
+ *                   The frequencies of the shared key part may come from the table as well.  With n14 > 0 (and n6 > 0) the launch also
+ *                   turns n6 values of each of off5 query heads by the same angles, n14 apart in the source rows from column off 3
+ *                   (no norm): in place, or into buf 6 [T, off5, n15] from column off 4 of each head.  f3 > 0: cosines and sines are multiplied by it.
  *                   With n11 > 0 the launch also keeps POOLED BLOCKS: row b of buf 5 (external [slots, n12, width]) becomes the mean of
  *                   the cached rows of positions b n11 .. b n11 + n11 - 1.  A step from position p leaves the blocks whose last
  *                   position is p - 1 .. p + T - 2 (a block is asked for at the earliest one position after its last).
- *                   buf 0 cache 1 src 2 ctl 3 norm weight 4 frequency table 5 pooled rows | off 0 src column 1 cache column 2 norm weight 3 query column
+ *                   buf 0 cache 1 src 2 ctl 3 norm weight 4 frequency table 5 pooled rows 6 turned query heads | off 0 src column 1 cache column 2 norm weight 3 query column
  *                   4 query weight 5 query heads 6 temperature period 7 frequency table offset
  *                   n 0 T 1 columns 2 src row stride 3 width 4 R 5 normed 6 rot 7 wdt 8 rotary layout 9 norm group 10 rotary inside the groups
- *                   11 positions per pooled block 12 pooled rows 13 order of norm and rotation
- *                   f 0 eps 1 rotary base 2 temperature coefficient
+ *                   11 positions per pooled block 12 pooled rows 13 order of norm and rotation 14 query head stride 15 its stride in buf 6
+ *                   f 0 eps 1 rotary base 2 temperature coefficient 3 rotary magnitude
  * CACHED_ATTENTION  softmax attention of the step's queries over cached keys and values.  A query row holds H * maps vectors
  *                   of dk (head h, map m at (h * maps + m) * dk); a key row G * maps vectors of dk; a value row G vectors of
  *                   dv; query (h, m) reads key (h / (H / G), m) and value h / (H / G).  The value cache may be the key cache
@@ -243,6 +255,8 @@ typedef enum ZgOpTag {
  *                   result is multiplied by sigmoid(gate[t, (h N + n) / group]) (the GATE op in the epilogue)
  *                   buf 0 dst 1 src 2 W 3 gate | off 0 W 1 src column 2 dst column 3 gate column 4 gate row stride
  *                   n 0 T 1 H 2 N 3 K 4 src head stride 5 src row stride 6 dst head stride 7 dst row stride 8 wdt 9 gate group
+ *                   10 outputs of the last head (0: N) 11 activation of the last head's outputs (as LINEAR's n6) 12 products that may
+ *                   round their inputs to bfloat16, as LINEAR's do (tensor cores; 0: exact) | f 0 activation parameter
  * POLY_NORM         dst[t] = a N(z) + b N(z^2) + c N(z^3) + e with N(v) = v / sqrt(mean(v^2) + f0) over the row, powers taken
  *                   element by element, (a, b, c, e) four weights; may run in place
  *                   buf 0 dst 1 src 2 coefficients | off 0 coefficients | n 0 T 1 columns 2 wdt | f 0 eps
@@ -280,7 +294,17 @@ typedef enum ZgOpTag {
  *                   buf 0 dst 1 u 2 gate logits 3 y 4 weights 5 state 6 ctl
  *                   off 0 u column 1 rl column 2 il column 3 y column 4 r_bias 5 i_bias 6 lam (weights)
  *                   n 0 T 1 W 2 u row stride 3 gate row stride 4 gate block width 5 gate block stride 6 y row stride
- *                   7 dst row stride 8 wdt 9 act of y | f 0 the constant in log a */
+ *                   7 dst row stride 8 wdt 9 act of y | f 0 the constant in log a
+ * STREAM_STEP       the residual step of a stack with s streams X_1 .. X_s (hyper-connections), closing a sublayer and opening the next in one
+ *                   launch.  Close (buf 2 given): X_b <- sum_a mix[a, b] X_a + f0 * out[b] * ls * y, all from the old streams, into buf 0.
+ *                   Open (buf 5 given): u = sum_a in[a] X_a of the new streams (of the old ones without a close);
+ *                   h = N(u) * f1, N a Dynamic Tanh (n5 = 8: w, b and alpha in a row) or nothing (n5 = 16).  With n6 > 0 h is token-shifted
+ *                   n6 times on its way out: row t of buf 5 holds n6 vectors h_t + (h_(t-1) - h_t) * mu_j, and the last row's h stays in
+ *                   the state buf 6 (external [slots, D], zeros for a fresh slot).
+ *                   buf 0 new streams [s, T, D] (without a close: buf 5 once more) 1 old streams 2 y 3 weights of the close 4 weights of the open 5 h [T, max(1, n6), D] 6 state 7 ctl
+ *                   off 0 out 1 mix [s, s] (from, to) 2 ls 3 in 4 norm 5 mu [n6, D]
+ *                   n 0 T 1 D 2 s 3 distance of the old streams (0: all equal, one [T, D]) 4 wdt 5 norm kind 6 shifts 7 ls given
+ *                   f 0 multiplier 1 gain of h */
 #define ZG_NO_BUF 0xFFFFFFFFu
 #define ZG_W_F32 0
 #define ZG_W_BF16 1

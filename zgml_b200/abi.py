@@ -23,12 +23,14 @@ OP_ALLREDUCE, OP_ALLGATHER = 12, 13   # multi-GPU extensions (need comm_init)
 (OP_TOKEN_SHIFT, OP_DEPTH_MIX, OP_ROTARY, OP_CACHE_APPEND, OP_CACHED_ATTENTION, OP_MAP_COMBINE, OP_GATE, OP_HEAD_LINEAR,
  OP_POLY_NORM) = range(22, 31)
 (OP_SSM_SCAN, OP_MIN_GRU, OP_GATED_NORM, OP_HEAD_NORM, OP_ACTIVATION, OP_RG_LRU) = range(31, 37)
-OP_END = 37
+OP_STREAM_STEP = 37
+OP_END = 38
 MASK_CAUSAL, MASK_WINDOW, MASK_BLOCK, MASK_POOLED = 0, 1, 2, 3      # pooled: a window, and one mean key and value per block before it
 NORM_LAYER, NORM_RMS, NORM_UNIT_OFFSET, NORM_GAIN = 0, 1, 2, 4
 NORM_DYNAMIC_TANH, NORM_NONE = 8, 16       # tanh(alpha x) w + b (bias and alpha follow w); the row itself: no statistics either way
 NORM_SCALAR_WEIGHT = 32                    # the weight is a single number for all columns
 DELTA_PLAIN, DELTA_SIGMOID_DECAY, DELTA_SILU_GATE, DELTA_OUT_SCALE, DELTA_HEAD_DECAY = 1, 2, 4, 8, 16     # forms of DELTA_RULE (n10)
+DELTA_BONUS, DELTA_EXP_DECAY, DELTA_WIDE_NORM = 32, 64, 128      # read before the write, with a bonus; exp(-exp(.)); a norm weight per head
 WEIGHTS_SOFTMAX, WEIGHTS_SIGMOID = 0, 1    # CACHED_ATTENTION: normalised over the visible keys, or sigmoid(score) of each
 ACTIVATIONS = {"relu2": 0, "silu": 1, "gelu_tanh": 2, "relu": 3, "softcap": 4, "gelu_erf": 5}     # "softcap": p * tanh(z / p), p the op's activation parameter
 NO_BUF = 0xFFFFFFFF

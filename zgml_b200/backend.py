@@ -207,23 +207,28 @@ class DeviceOp:
         return o
 
     @staticmethod
-    def embed(dst, ctl, table, table_off, T, D, scale, wdt, positions_off=None, bigram=None):
+    def embed(dst, ctl, table, table_off, T, D, scale, wdt, positions_off=None, bigram=None, dyt_off=None):
         """Rows of the table times `scale`; with `positions_off` a learned position row of the same arena is added, unscaled.
         `bigram` = (offset, buckets, mul_prev, mul_cur): a row of that table (buckets + 1 rows in the same arena) is added, unscaled, at
-        (previous token * mul_prev + token * mul_cur) mod buckets; a sequence's first token takes the last row."""
+        (previous token * mul_prev + token * mul_cur) mod buckets; a sequence's first token takes the last row.
+        `dyt_off`: the row then passes a Dynamic Tanh whose weight, bias and alpha lie there."""
         b_off, buckets, mul_prev, mul_cur = bigram or (0, 0, 0, 0)
         if buckets:
             mul_prev, mul_cur = mul_prev % buckets, mul_cur % buckets       # the same residues, and the products fit the kernel's integers
-        return DeviceOp._seq(abi.OP_EMBED, [dst, ctl, table], [table_off, positions_off or 0, b_off], [T, D, wdt, int(positions_off is not None), buckets, mul_prev, mul_cur], [scale])
+        return DeviceOp._seq(abi.OP_EMBED, [dst, ctl, table], [table_off, positions_off or 0, b_off, dyt_off or 0],
+                             [T, D, wdt, int(positions_off is not None), buckets, mul_prev, mul_cur, int(dyt_off is not None)], [scale])
 
     @staticmethod
     def linear(dst, src, w, w_off, M, N, K, wdt, bias=None, bias_off=0, src_off=0, dst_off=0, src_rs=0, dst_rs=0, act=None, act_param=0.0, ctl=None, src_slot_stride=0,
-               act_cols=None):
+               act_cols=None, pairs=False, live_rows=0):
         """`act`: an activation of abi.ACTIVATIONS applied in the epilogue, after the bias (`act_param`: its parameter, where it has one), to
         the output columns act_cols = (first, end) only, where given.
-        `src_slot_stride` > 0: the source rows are the slot's part of a per-sequence state buffer (that many elements per slot; slot from `ctl`)."""
+        `src_slot_stride` > 0: the source rows are the slot's part of a per-sequence state buffer (that many elements per slot; slot from `ctl`);
+        with `live_rows` rows from position + live_rows on are not computed.  `pairs`: W holds 2 N rows, a gate row and the row it multiplies in
+        turns, dst = act(gate) * up."""
         return DeviceOp._seq(abi.OP_LINEAR, [dst, src, w, bias, ctl if src_slot_stride else None], [w_off, bias_off, src_off, dst_off],
-                             [M, N, K, src_rs or K, dst_rs or N, wdt, 0 if act is None else abi.ACTIVATIONS[act] + 1, src_slot_stride] + list(act_cols or ()), [act_param])
+                             [M, N, K, src_rs or K, dst_rs or N, wdt, 0 if act is None else abi.ACTIVATIONS[act] + 1, src_slot_stride] + list(act_cols or (0, 0)) +
+                             [int(pairs), live_rows], [act_param])
 
     @staticmethod
     def norm(dst, src, w, w_off, rows, cols, eps, wdt, kind="layer", res=None, then=None, then_w=None, then_w_off=0, then_kind="layer",
@@ -279,26 +284,28 @@ class DeviceOp:
     @staticmethod
     def delta_rule(dst, qkv, beta, a, gate, w, state, ctl, q_off, k_off, v_off, beta_off, a_log_off, dt_bias_off, norm_off,
                    T, H, G, dim, vdim, qkv_rs, beta_rs, a_rs, gate_rs, wdt, norm_eps, unit_eps, q_scale, gate_off=0, plain=False, decay_tau=None,
-                   silu_gate=False, out_scale=None, dst_rs=0, dst_col=0, head_decay=False, a_col=0):
+                   silu_gate=False, out_scale=None, dst_rs=0, dst_col=0, head_decay=False, a_col=0, bonus_off=None, exp_decay=False, wide_norm=False):
         """`plain`: no unit vectors and no correction by the state (S <- g S + k v^T: gated linear attention; `beta` may be None).
         `decay_tau`: the decay is sigmoid(a + dt_bias)^(1 / tau) instead of exp(-exp(A_log) softplus(a + dt_bias)).  `silu_gate`: the
         output gate is silu instead of sigmoid.  `head_decay`: one decay per head (rows of `a` and dt_bias hold H values).  `out_scale` multiplies the result, which may land at column `dst_col` of rows
-        `dst_rs` wide."""
+        `dst_rs` wide.  `bonus_off` (with `plain`): the state is read before the token's write, and the token joins through a bonus per head and key
+        channel (H * dim weights there).  `exp_decay`: the decay is exp(-exp(a + dt_bias)).  `wide_norm`: the norm weight holds H * vdim values."""
         form = (abi.DELTA_PLAIN if plain else 0) | (abi.DELTA_SIGMOID_DECAY if decay_tau is not None else 0) | (abi.DELTA_SILU_GATE if silu_gate else 0) | \
-            (abi.DELTA_OUT_SCALE if out_scale is not None else 0) | (abi.DELTA_HEAD_DECAY if head_decay else 0)
+            (abi.DELTA_OUT_SCALE if out_scale is not None else 0) | (abi.DELTA_HEAD_DECAY if head_decay else 0) | \
+            (abi.DELTA_BONUS if bonus_off is not None else 0) | (abi.DELTA_EXP_DECAY if exp_decay else 0) | (abi.DELTA_WIDE_NORM if wide_norm else 0)
         return DeviceOp._seq(abi.OP_DELTA_RULE, [dst, qkv, beta, a, gate, w, state, ctl],
                              [q_off, k_off, v_off, beta_off, a_log_off, dt_bias_off, norm_off, gate_off],
-                             [T, H, G, dim, vdim, qkv_rs, beta_rs, a_rs, gate_rs, wdt, form, dst_rs, dst_col, a_col], [norm_eps, unit_eps, q_scale, decay_tau or 0.0, out_scale or 0.0])
+                             [T, H, G, dim, vdim, qkv_rs, beta_rs, a_rs, gate_rs, wdt, form, dst_rs, dst_col, a_col, bonus_off or 0], [norm_eps, unit_eps, q_scale, decay_tau or 0.0, out_scale or 0.0])
 
     @staticmethod
-    def route(dst, logits, w, corr_off, T, n_outputs, top, wdt, logits_off=0, logits_rs=0, mode="corrected_softmax", groups=0, groups_kept=0):
+    def route(dst, logits, w, corr_off, T, n_outputs, top, wdt, logits_off=0, logits_rs=0, mode="corrected_softmax", groups=0, groups_kept=0, scale=1.0):
         """mode "corrected_softmax": softmax over all outputs, choice by softmax + correction, weights not renormalised;
         "biased_top": choice by logits + bias, weights = softmax over the chosen biased logits; "corrected_sigmoid": sigmoid
         scores, choice by score + correction among the outputs of the `groups_kept` best of `groups` equal groups (a group scores
-        the sum of its two largest choice scores), weights = the chosen scores divided by their sum."""
+        the sum of its two largest choice scores), weights = the chosen scores divided by their sum; "scaled_sigmoid": the same choice, weights = the chosen scores times `scale`."""
         return DeviceOp._seq(abi.OP_ROUTE, [dst, logits, w], [corr_off, logits_off],
-                             [T, n_outputs, top, logits_rs or n_outputs, wdt, {"corrected_softmax": 0, "biased_top": 1, "corrected_sigmoid": 2}[mode],
-                              groups, groups_kept])
+                             [T, n_outputs, top, logits_rs or n_outputs, wdt, {"corrected_softmax": 0, "biased_top": 1, "corrected_sigmoid": 2, "scaled_sigmoid": 3}[mode],
+                              groups, groups_kept], [scale])
 
     @staticmethod
     def moe_ffn(dst, src, route, w, scratch, gate_off, up_off, down_off, T, D, ff, experts, top, wdt, limit, alpha, up_offset=1.0):
@@ -322,19 +329,27 @@ class DeviceOp:
     @staticmethod
     def cache_append(cache, src, ctl, src_col, cache_col, T, cols, src_rs, width, rows, norm_w=None, norm_off=0, normed=0, eps=0.0, wdt=0,
                      rot=0, rot_base=0.0, rot_layout="pairs", norm_group=0, q_heads=0, q_col=0, q_norm_off=0, temp_coef=0.0, temp_every=0, head_rot=0,
-                     freqs=None, freqs_off=0, order="rotate_norm", pooled=None, pool=0, pool_rows=0):
+                     freqs=None, freqs_off=0, order="rotate_norm", pooled=None, pool=0, pool_rows=0,
+                     rot_scale=0.0, turned_heads=None):
         """`norm_group` > 0: the normed columns are normed in groups of that many (key heads) sharing one weight of that size.
         `q_heads` > 0: that many query heads of norm_group values at column q_col of the source rows are normed in place by the same
         launch (weight at q_norm_off of norm_w's arena), times the position-dependent temperature of HEAD_NORM.
         `head_rot` > 0: every normed group (key and query heads) is first turned by the token's rotary position on its first head_rot
         values (`rot_layout`; frequencies from `rot_base`, or from the f32 table `freqs` at element `freqs_off`), then normed;
         `order` "norm_rotate": normed and weighted first, then turned; "rotate": turned and not normed (norm_w may be None).
-        `pool` > 0: row b of `pooled` (`pool_rows` rows per slot) becomes the mean of the cached rows of block b of `pool` positions."""
+        `pool` > 0: row b of `pooled` (`pool_rows` rows per slot) becomes the mean of the cached rows of block b of `pool` positions.
+        `rot_scale` > 0 multiplies cosines and sines.  `turned_heads` = (heads, column, stride, destination, its column, its stride): with `rot` the same
+        launch turns `rot` values of that many query heads, `stride` apart in the source rows from `column` on, in place (destination None) or
+        into rows of heads * its-stride values."""
+        if turned_heads:
+            q_heads, q_col, q_hs, q_dst, q_norm_off, q_dst_hs = turned_heads
+        else:
+            q_hs, q_dst, q_dst_hs = 0, None, 0
         orders = {"rotate_norm": abi.ROTATE_THEN_NORM, "norm_rotate": abi.NORM_THEN_ROTATE, "rotate": abi.ROTATE_ONLY}
-        return DeviceOp._seq(abi.OP_CACHE_APPEND, [cache, src, ctl, norm_w if normed else None, freqs if head_rot else None, pooled if pool else None],
+        return DeviceOp._seq(abi.OP_CACHE_APPEND, [cache, src, ctl, norm_w if normed else None, freqs if head_rot or rot else None, pooled if pool else None, q_dst],
                              [src_col, cache_col, norm_off, q_col, q_norm_off, q_heads, temp_every, freqs_off],
-                             [T, cols, src_rs, width, rows, normed, rot, wdt, {"pairs": 0, "halves": 1}[rot_layout], norm_group, head_rot, pool, pool_rows, orders[order]],
-                             [eps, rot_base, temp_coef])
+                             [T, cols, src_rs, width, rows, normed, rot, wdt, {"pairs": 0, "halves": 1}[rot_layout], norm_group, head_rot, pool, pool_rows, orders[order], q_hs,
+                              q_dst_hs], [eps, rot_base, temp_coef, rot_scale])
 
     @staticmethod
     def cached_attention(dst, q, k_cache, v_cache, ctl, q_col, k_col, v_col, T, H, G, maps, dk, dv, q_rs, k_width, v_width, rows, scale,
@@ -362,9 +377,12 @@ class DeviceOp:
 
     @staticmethod
     def head_linear(dst, src, w, w_off, T, H, N, K, wdt, src_col=0, src_hs=0, src_rs=0, dst_col=0, dst_hs=0, dst_rs=0, gate=None, gate_col=0, gate_rs=0,
-                    gate_group=1):
+                    gate_group=1, n_last=0, last_act=None, last_act_param=0.0, rounded=False):
+        """`n_last`: outputs of the last head, where they are not N; `last_act`: an activation they alone pass; `rounded`: the products may round
+        their inputs to bfloat16 (many rows of a bfloat16 session then run on the tensor cores, as LINEAR's do)."""
         return DeviceOp._seq(abi.OP_HEAD_LINEAR, [dst, src, w, gate], [w_off, src_col, dst_col, gate_col, gate_rs],
-                             [T, H, N, K, src_hs or K, src_rs or H * K, dst_hs or N, dst_rs or H * N, wdt, gate_group if gate is not None else 0])
+                             [T, H, N, K, src_hs or K, src_rs or H * K, dst_hs or N, dst_rs or H * N, wdt, gate_group if gate is not None else 0,
+                              n_last, 0 if last_act is None else abi.ACTIVATIONS[last_act] + 1, int(rounded)], [last_act_param])
 
     @staticmethod
     def poly_norm(dst, src, w, coeff_off, T, cols, eps, wdt):
@@ -402,6 +420,17 @@ class DeviceOp:
         c % gate_bw of a `gates` row, from r_col and i_col; biases and `lam` are weights; `y_act` is applied to y on its way out."""
         return DeviceOp._seq(abi.OP_RG_LRU, [dst, u, gates, y, w, state, ctl], [u_col, r_col, i_col, y_col, r_bias_off, i_bias_off, lam_off],
                              [T, W, u_rs, gate_rs, gate_bw, gate_bs, y_rs, dst_rs or W, wdt, 0 if y_act is None else abi.ACTIVATIONS[y_act] + 1], [rate])
+
+
+    @staticmethod
+    def stream_step(T, D, streams, wdt, dst=None, src=None, src_stride=0, y=None, close_w=None, out_off=0, mix_off=0, ls_off=None, mult=1.0,
+                    h=None, open_w=None, in_off=0, kind="dyt", norm_off=0, gain=1.0, shifts=0, mu_off=0, state=None, ctl=None):
+        """Residual step of a stack with several streams.  With `y`: every new stream is a mixture of the old ones (mix [from, to]) plus
+        mult * out[stream] * ls * y.  With `h`: in-weighted sum of the streams, normed ("dyt": Dynamic Tanh, "none"), times `gain`, token-shifted
+        `shifts` times (mu [shifts, D], carried row `state`) on its way out."""
+        return DeviceOp._seq(abi.OP_STREAM_STEP, [dst if y is not None else h, src, y, close_w if y is not None else None, open_w if h is not None else None, h,
+                                                  state if shifts else None, ctl if shifts else None], [out_off, mix_off, ls_off or 0, in_off, norm_off, mu_off],
+                             [T, D, streams, src_stride, wdt, {"dyt": abi.NORM_DYNAMIC_TANH, "none": abi.NORM_NONE}[kind], shifts, int(ls_off is not None)], [mult, gain])
 
 
 @dataclass

@@ -72,10 +72,15 @@ __device__ __forceinline__ uint64_t make_desc(uint32_t smem_addr) {
 
 // f32 rows -> dense bf16 [Mp][Kp] (zero padding), two k per thread
 // (ctl: the rows are those of a per-sequence state buffer, `slot_stride` elements per slot; the slot is the control word's)
+// (rows_from > 0: rows from position + rows_from on are not wanted, up to the end of their 128-row tile)
+// blockIdx.z: a batch of sources x_hs apart, each with its own padded rows in `out`
 __global__ void k_to_bf16(const float* __restrict__ x, uint32_t x_rs, uint32_t* __restrict__ out, uint32_t kp2, uint32_t M, uint32_t K, const float* __restrict__ ctl,
-                          uint32_t slot_stride) {
-    if (ctl) x += (size_t)reinterpret_cast<const int*>(ctl)[ZG_CTL_SLOT] * slot_stride;
+                          uint32_t slot_stride, uint32_t rows_from, uint32_t x_hs) {
     const uint32_t m = blockIdx.y;
+    if (rows_from && m / BM * BM >= (uint32_t)reinterpret_cast<const int*>(ctl)[ZG_CTL_POS] + rows_from) return;
+    if (ctl) x += (size_t)reinterpret_cast<const int*>(ctl)[ZG_CTL_SLOT] * slot_stride;
+    x += (size_t)blockIdx.z * x_hs;
+    out += (size_t)blockIdx.z * gridDim.y * kp2;
     for (uint32_t k2 = blockIdx.x * blockDim.x + threadIdx.x; k2 < kp2; k2 += gridDim.x * blockDim.x) {
         const uint32_t k = 2 * k2;
         const float a = (m < M && k < K) ? x[(size_t)m * x_rs + k] : 0.0f;
@@ -113,15 +118,27 @@ struct GemmParams {
     uint32_t act;            // applied after the bias: 0 none, 1 relu^2, 2 silu, 3 gelu (tanh form), 4 relu, 5 smooth cap act_p * tanh(z / act_p), 6 gelu (erf form)
     float act_p;
     uint32_t act_lo, act_hi; // the columns it applies to
-    const int* tile_group;   // GROUPED: weight matrix (third TMA coordinate) of every 128-row tile, -1: tile unused
+    const int* tile_group;   // kGrouped: weight matrix (third TMA coordinate) of every 128-row tile, -1: tile unused
+    const int* ctl;          // kPlain with rows_from: tiles from row position + rows_from on are skipped
+    uint32_t rows_from;
+    uint32_t heads, n_last, a_rows, out_hs;   // kBatched: heads, rows of the last head's matrix, padded source rows per head, columns between the heads' outputs
 };
 
-// GROUPED: the rows are sorted by weight matrix (expert) in whole 128-row tiles; tile t multiplies with matrix tile_group[t]
+// kGrouped: the rows are sorted by weight matrix (expert) in whole 128-row tiles; tile t multiplies with matrix tile_group[t]
 // of the stacked [groups][N][K] weight tensor.
-template <bool GROUPED, int ACT>        // ACT: the activation of the epilogue (GemmParams::act; one instantiation each)
+// kBatched: blockIdx.z names a head with source rows, weight rows and output columns of its own (all in one tensor each).  A tile at the
+// end of a head reads on into the next head's weight rows; those columns are not written.
+// PAIRS: weight rows 2n and 2n + 1 are a gate and what it multiplies: out[., n] = act(gate) * up.
+enum { kPlain = 0, kGrouped = 1, kBatched = 2 };
+template <int MODE, int ACT, bool PAIRS>        // ACT: the activation of the epilogue (GemmParams::act; one instantiation each)
 __global__ void __launch_bounds__(kThreads, 1)
 dense_gemm_kernel(const __grid_constant__ CUtensorMap tmap_a, const __grid_constant__ CUtensorMap tmap_b, const GemmParams p) {
+    constexpr bool GROUPED = MODE == kGrouped;
     int group = 0;
+    const uint32_t head = MODE == kBatched ? blockIdx.z : 0, N = MODE == kBatched && head + 1 == p.heads ? p.n_last : p.N;
+    if (MODE == kBatched && blockIdx.x * BN >= N) return;
+    if (MODE == kPlain && p.rows_from && blockIdx.y * BM >= (uint32_t)p.ctl[ZG_CTL_POS] + p.rows_from) return;
+    float* const outp = p.out + (MODE == kBatched ? (size_t)head * p.out_hs : 0);
     if (GROUPED) {
         group = p.tile_group[blockIdx.y];
         if (group < 0) return;   // uniform over the CTA, before any barrier or TMEM allocation
@@ -155,9 +172,9 @@ dense_gemm_kernel(const __grid_constant__ CUtensorMap tmap_a, const __grid_const
                 const uint32_t s = kt % kStages, ph = (kt / kStages) & 1;
                 if (!mbar_wait(empty + 8 * s, ph ^ 1)) break;
                 mbar_expect_tx(full + 8 * s, kStage);
-                tma_load_2d(base + s * kStage, &tmap_a, kt * BK, tile_m * BM, full + 8 * s);
+                tma_load_2d(base + s * kStage, &tmap_a, kt * BK, head * p.a_rows + tile_m * BM, full + 8 * s);
                 if (GROUPED) tma_load_3d(base + s * kStage + kTileA, &tmap_b, kt * BK, tile_n * BN, (uint32_t)group, full + 8 * s);
-                else tma_load_2d(base + s * kStage + kTileA, &tmap_b, kt * BK, tile_n * BN, full + 8 * s);
+                else tma_load_2d(base + s * kStage + kTileA, &tmap_b, kt * BK, head * p.N + tile_n * BN, full + 8 * s);
             }
         }
     } else if (warp == 1) {
@@ -209,14 +226,30 @@ dense_gemm_kernel(const __grid_constant__ CUtensorMap tmap_a, const __grid_const
             for (int i = 0; i < 8; i++) tb[lane * 9 + i] = make_uint4(v[4 * i], v[4 * i + 1], v[4 * i + 2], v[4 * i + 3]);
             __syncwarp();
             const uint32_t n0 = tile_n * BN + c0;
-            const bool some = ACT && n0 < p.act_hi && n0 + 32 > p.act_lo;     // uniform: whether any of these columns takes the activation
+            const bool acts = ACT && (MODE != kBatched || head + 1 == p.heads), some = acts && n0 < p.act_hi && n0 + 32 > p.act_lo;     // uniform: whether any of these columns takes the activation
             auto finish = [&](float z, uint32_t n) {
                 if (!ACT) return z;
                 const float a = gemm_act<ACT>(z, p.act_p);
-                return n >= p.act_lo && n < p.act_hi ? a : z;
+                return acts && n >= p.act_lo && n < p.act_hi ? a : z;
             };
-            if (n0 < p.N) {
-                if (p.out_vec4 && n0 + 32 <= p.N) {
+            if (PAIRS) {
+                if (p.out_vec4 && n0 + 32 <= N) {
+                    const uint32_t nn = n0 + 4 * (lane & 7);
+#pragma unroll
+                    for (int it = 0; it < 8; it++) {
+                        const uint32_t rr = it * 4 + (lane >> 3), mm = m_base + rr;
+                        const uint4 o = tb[rr * 9 + (lane & 7)];
+                        const float2 f = make_float2(gemm_act<ACT>(__uint_as_float(o.x), p.act_p) * __uint_as_float(o.y), gemm_act<ACT>(__uint_as_float(o.z), p.act_p) * __uint_as_float(o.w));
+                        if (mm < p.M) *reinterpret_cast<float2*>(outp + (size_t)mm * p.out_rs + nn / 2) = f;
+                    }
+                } else if (lane < 16 && n0 + 2 * lane + 1 < N) {
+                    const uint32_t* tw = reinterpret_cast<const uint32_t*>(tb);
+                    for (int rr = 0; rr < 32; rr++)
+                        if (m_base + rr < p.M)
+                            outp[(size_t)(m_base + rr) * p.out_rs + n0 / 2 + lane] = gemm_act<ACT>(__uint_as_float(tw[rr * 36 + 2 * lane]), p.act_p) * __uint_as_float(tw[rr * 36 + 2 * lane + 1]);
+                }
+            } else if (n0 < N) {
+                if (p.out_vec4 && n0 + 32 <= N) {
                     const uint32_t nn = n0 + 4 * (lane & 7);
                     float b[4] = {0.0f, 0.0f, 0.0f, 0.0f};
                     if (p.bias) for (int j = 0; j < 4; j++) b[j] = __bfloat162float(p.bias[nn + j]);
@@ -227,7 +260,7 @@ dense_gemm_kernel(const __grid_constant__ CUtensorMap tmap_a, const __grid_const
                         const uint4 o = tb[rr * 9 + (lane & 7)];
                         const float4 f = make_float4(finish(__uint_as_float(o.x) + b[0], nn), finish(__uint_as_float(o.y) + b[1], nn + 1), finish(__uint_as_float(o.z) + b[2], nn + 2),
                                                      finish(__uint_as_float(o.w) + b[3], nn + 3));
-                        if (mm < p.M) *reinterpret_cast<float4*>(p.out + (size_t)mm * p.out_rs + nn) = f;
+                        if (mm < p.M) *reinterpret_cast<float4*>(outp + (size_t)mm * p.out_rs + nn) = f;
                     }
                     } else {
 #pragma unroll
@@ -235,14 +268,14 @@ dense_gemm_kernel(const __grid_constant__ CUtensorMap tmap_a, const __grid_const
                         const uint32_t rr = it * 4 + (lane >> 3), mm = m_base + rr;
                         const uint4 o = tb[rr * 9 + (lane & 7)];
                         const float4 f = make_float4(__uint_as_float(o.x) + b[0], __uint_as_float(o.y) + b[1], __uint_as_float(o.z) + b[2], __uint_as_float(o.w) + b[3]);
-                        if (mm < p.M) *reinterpret_cast<float4*>(p.out + (size_t)mm * p.out_rs + nn) = f;
+                        if (mm < p.M) *reinterpret_cast<float4*>(outp + (size_t)mm * p.out_rs + nn) = f;
                     }
                     }
-                } else if (n0 + lane < p.N) {
+                } else if (n0 + lane < N) {
                     const uint32_t* tw = reinterpret_cast<const uint32_t*>(tb);
                     const float b = p.bias ? __bfloat162float(p.bias[n0 + lane]) : 0.0f;
                     for (int rr = 0; rr < 32; rr++)
-                        if (m_base + rr < p.M) p.out[(size_t)(m_base + rr) * p.out_rs + n0 + lane] = finish(__uint_as_float(tw[rr * 36 + lane]) + b, n0 + lane);
+                        if (m_base + rr < p.M) outp[(size_t)(m_base + rr) * p.out_rs + n0 + lane] = finish(__uint_as_float(tw[rr * 36 + lane]) + b, n0 + lane);
                 }
             }
             __syncwarp();
@@ -260,8 +293,14 @@ EncodeTiledFn g_encode = nullptr;
 bool g_attr_set = false;
 constexpr int kActs = 7;
 typedef void (*GemmKernel)(const CUtensorMap, const CUtensorMap, const GemmParams);
-const GemmKernel g_kernel[kActs] = {dense_gemm_kernel<false, 0>, dense_gemm_kernel<false, 1>, dense_gemm_kernel<false, 2>, dense_gemm_kernel<false, 3>,
-                                    dense_gemm_kernel<false, 4>, dense_gemm_kernel<false, 5>, dense_gemm_kernel<false, 6>};   // by activation
+#define ZG_ACTS(MODE_, PAIRS_)                                                                                                                           \
+    {dense_gemm_kernel<MODE_, 0, PAIRS_>, dense_gemm_kernel<MODE_, 1, PAIRS_>, dense_gemm_kernel<MODE_, 2, PAIRS_>, dense_gemm_kernel<MODE_, 3, PAIRS_>, \
+     dense_gemm_kernel<MODE_, 4, PAIRS_>, dense_gemm_kernel<MODE_, 5, PAIRS_>, dense_gemm_kernel<MODE_, 6, PAIRS_>}
+const GemmKernel g_kernel[2][kActs] = {ZG_ACTS(kPlain, false), ZG_ACTS(kPlain, true)};   // [pairs][activation]
+#undef ZG_ACTS
+GemmKernel batched_kernel(uint32_t act) {      // the activations a batched product's last head can have
+    return act == 0 ? dense_gemm_kernel<kBatched, 0, false> : act == 5 ? dense_gemm_kernel<kBatched, 5, false> : (GemmKernel)nullptr;
+}
 
 bool prepare() {
     if (!g_encode) {
@@ -274,8 +313,9 @@ bool prepare() {
         g_encode = (EncodeTiledFn)fn;
     }
     if (!g_attr_set) {
-        cudaError_t e = cudaFuncSetAttribute(dense_gemm_kernel<true, 0>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)kSmem);
-        for (int k = 0; k < kActs && e == cudaSuccess; k++) e = cudaFuncSetAttribute(g_kernel[k], cudaFuncAttributeMaxDynamicSharedMemorySize, (int)kSmem);
+        cudaError_t e = cudaFuncSetAttribute(dense_gemm_kernel<kGrouped, 0, false>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)kSmem);
+        for (int k = 0; k < 2 * kActs && e == cudaSuccess; k++) e = cudaFuncSetAttribute(g_kernel[k / kActs][k % kActs], cudaFuncAttributeMaxDynamicSharedMemorySize, (int)kSmem);
+        for (uint32_t k = 0; k < 6 && e == cudaSuccess; k += 5) e = cudaFuncSetAttribute(batched_kernel(k), cudaFuncAttributeMaxDynamicSharedMemorySize, (int)kSmem);
         if (e != cudaSuccess) { zg_set_error("cudaFuncSetAttribute(dense_gemm) failed: %s", cudaGetErrorString(e)); return false; }
         g_attr_set = true;
     }
@@ -299,11 +339,13 @@ unsigned int zg_dense_gemm_timeouts() {
 }
 
 bool zg_dense_gemm_launch(const void* w_bf16, const void* bias_bf16, const float* src, float* dst, uint32_t M, uint32_t N, uint32_t K,
-                          uint32_t src_rs, uint32_t dst_rs, float* scratch, cudaStream_t st, uint32_t act, float act_p, uint32_t act_lo, uint32_t act_hi, const float* ctl, uint32_t slot_stride) {
+                          uint32_t src_rs, uint32_t dst_rs, float* scratch, cudaStream_t st, uint32_t act, float act_p, uint32_t act_lo, uint32_t act_hi, const float* ctl, uint32_t slot_stride, bool pairs,
+                          uint32_t rows_from) {
     if (!prepare()) return false;
+    if (pairs) N *= 2;                                   // weight rows
     const uint32_t Kp = (K + BK - 1) / BK * BK, Mp = (M + BM - 1) / BM * BM;
     uint32_t* xb = reinterpret_cast<uint32_t*>(scratch);
-    k_to_bf16<<<dim3((Kp / 2 + 255) / 256, Mp), 256, 0, st>>>(src, src_rs, xb, Kp / 2, M, K, ctl, slot_stride);
+    k_to_bf16<<<dim3((Kp / 2 + 255) / 256, Mp), 256, 0, st>>>(src, src_rs, xb, Kp / 2, M, K, ctl, slot_stride, rows_from, 0u);
     ZG_COUNT_LAUNCH();
     CUtensorMap map_a, map_b;
     const cuuint32_t estr[2] = {1, 1};
@@ -323,13 +365,14 @@ bool zg_dense_gemm_launch(const void* w_bf16, const void* bias_bf16, const float
                               CU_TENSOR_MAP_SWIZZLE_128B, CU_TENSOR_MAP_L2_PROMOTION_L2_256B, CU_TENSOR_MAP_FLOAT_OOB_FILL_NONE);
         if (r != CUDA_SUCCESS) { zg_set_error("cuTensorMapEncodeTiled(weights) failed (%d)", (int)r); return false; }
     }
-    GemmParams p;
+    GemmParams p = {};
+    p.ctl = reinterpret_cast<const int*>(ctl); p.rows_from = rows_from;
     p.out = dst; p.bias = reinterpret_cast<const __nv_bfloat16*>(bias_bf16); p.M = M; p.N = N; p.K = K; p.out_rs = dst_rs; p.act = act; p.act_p = act_p; p.act_lo = act_lo; p.act_hi = act_hi;
     p.out_vec4 = ((reinterpret_cast<uintptr_t>(dst) & 15) == 0 && (dst_rs & 3) == 0) ? 1u : 0u;
     p.tile_group = nullptr;
     dim3 grid((N + BN - 1) / BN, (M + BM - 1) / BM);
     if (act >= (uint32_t)kActs) { zg_set_error("dense gemm: unknown activation %u", act); return false; }
-    g_kernel[act]<<<grid, kThreads, kSmem, st>>>(map_a, map_b, p);
+    g_kernel[pairs ? 1 : 0][act]<<<grid, kThreads, kSmem, st>>>(map_a, map_b, p);
     ZG_COUNT_LAUNCH();
     cudaError_t e = cudaGetLastError();
     if (e != cudaSuccess) { zg_set_error("dense gemm launch failed: %s", cudaGetErrorString(e)); return false; }
@@ -358,14 +401,48 @@ bool zg_dense_gemm_grouped_launch(const void* w_bf16, uint32_t groups, const voi
                               CU_TENSOR_MAP_SWIZZLE_128B, CU_TENSOR_MAP_L2_PROMOTION_L2_256B, CU_TENSOR_MAP_FLOAT_OOB_FILL_NONE);
         if (r != CUDA_SUCCESS) { zg_set_error("cuTensorMapEncodeTiled(stacked weights) failed (%d)", (int)r); return false; }
     }
-    GemmParams p;
+    GemmParams p = {};
     p.out = dst; p.bias = nullptr; p.M = rows; p.N = N; p.K = K; p.out_rs = dst_rs; p.act = 0; p.act_p = 0.0f; p.act_lo = p.act_hi = 0;
     p.out_vec4 = ((reinterpret_cast<uintptr_t>(dst) & 15) == 0 && (dst_rs & 3) == 0) ? 1u : 0u;
     p.tile_group = d_tile_group;
     dim3 grid((N + BN - 1) / BN, rows / BM);
-    dense_gemm_kernel<true, 0><<<grid, kThreads, kSmem, st>>>(map_a, map_b, p);
+    dense_gemm_kernel<kGrouped, 0, false><<<grid, kThreads, kSmem, st>>>(map_a, map_b, p);
     ZG_COUNT_LAUNCH();
     cudaError_t e = cudaGetLastError();
     if (e != cudaSuccess) { zg_set_error("grouped dense gemm launch failed: %s", cudaGetErrorString(e)); return false; }
+    return true;
+}
+
+bool zg_dense_gemm_batched_usable(uint32_t M, uint32_t N, uint32_t K, uint32_t act) { return M > 8 && N >= 8 && K >= 64 && K % 8 == 0 && batched_kernel(act) != nullptr; }
+size_t zg_dense_gemm_batched_scratch_elems(uint32_t heads, uint32_t M, uint32_t K) { return (size_t)heads * zg_dense_gemm_scratch_elems(M, K); }
+bool zg_dense_gemm_batched_launch(const void* w_bf16, const float* src, float* dst, uint32_t heads, uint32_t M, uint32_t N, uint32_t n_last, uint32_t K, uint32_t src_hs, uint32_t src_rs,
+                                  uint32_t dst_hs, uint32_t dst_rs, float* scratch, cudaStream_t st, uint32_t act_last, float act_p) {
+    if (!prepare()) return false;
+    const uint32_t Kp = (K + BK - 1) / BK * BK, Mp = (M + BM - 1) / BM * BM;
+    uint32_t* xb = reinterpret_cast<uint32_t*>(scratch);
+    k_to_bf16<<<dim3((Kp / 2 + 255) / 256, Mp, heads), 256, 0, st>>>(src, src_rs, xb, Kp / 2, M, K, (const float*)nullptr, 0u, 0u, src_hs);
+    ZG_COUNT_LAUNCH();
+    CUtensorMap map_a, map_b;
+    const cuuint32_t estr[2] = {1, 1};
+    const cuuint64_t adim[2] = {Kp, (cuuint64_t)heads * Mp}, astride[1] = {(cuuint64_t)Kp * 2};
+    const cuuint32_t abox[2] = {BK, BM};
+    CUresult r = g_encode(&map_a, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 2, xb, adim, astride, abox, estr, CU_TENSOR_MAP_INTERLEAVE_NONE, CU_TENSOR_MAP_SWIZZLE_128B,
+                          CU_TENSOR_MAP_L2_PROMOTION_L2_128B, CU_TENSOR_MAP_FLOAT_OOB_FILL_NONE);
+    if (r != CUDA_SUCCESS) { zg_set_error("cuTensorMapEncodeTiled(batched rows) failed (%d)", (int)r); return false; }
+    const cuuint64_t bdim[2] = {K, (cuuint64_t)(heads - 1) * N + n_last}, bstride[1] = {(cuuint64_t)K * 2};
+    const cuuint32_t bbox[2] = {BK, BN};
+    r = g_encode(&map_b, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 2, const_cast<void*>(w_bf16), bdim, bstride, bbox, estr, CU_TENSOR_MAP_INTERLEAVE_NONE, CU_TENSOR_MAP_SWIZZLE_128B,
+                 CU_TENSOR_MAP_L2_PROMOTION_L2_256B, CU_TENSOR_MAP_FLOAT_OOB_FILL_NONE);
+    if (r != CUDA_SUCCESS) { zg_set_error("cuTensorMapEncodeTiled(batched weights) failed (%d)", (int)r); return false; }
+    GemmParams p = {};
+    p.out = dst; p.M = M; p.N = N; p.K = K; p.out_rs = dst_rs; p.act = act_last; p.act_p = act_p; p.act_lo = 0; p.act_hi = 0xffffffffu;
+    p.heads = heads; p.n_last = n_last; p.a_rows = Mp; p.out_hs = dst_hs;
+    p.out_vec4 = ((reinterpret_cast<uintptr_t>(dst) & 15) == 0 && (dst_rs & 3) == 0 && (dst_hs & 3) == 0) ? 1u : 0u;
+    GemmKernel kernel = batched_kernel(act_last);
+    if (!kernel) { zg_set_error("batched dense gemm: activation %u", act_last); return false; }
+    kernel<<<dim3(((N > n_last ? N : n_last) + BN - 1) / BN, Mp / BM, heads), kThreads, kSmem, st>>>(map_a, map_b, p);
+    ZG_COUNT_LAUNCH();
+    cudaError_t e = cudaGetLastError();
+    if (e != cudaSuccess) { zg_set_error("batched dense gemm launch failed: %s", cudaGetErrorString(e)); return false; }
     return true;
 }

@@ -7,6 +7,7 @@
 #include "seq_common.cuh"
 
 #include <math.h>
+#include <stdlib.h>
 
 namespace {
 
@@ -93,14 +94,15 @@ template <typename WT>
 __global__ void k_cache_append(float* __restrict__ cache, const float* __restrict__ src, const float* __restrict__ ctl, const WT* __restrict__ nw_,
                                uint32_t cols, uint32_t src_rs, uint32_t width, uint32_t R, uint32_t normed, uint32_t rot, uint32_t layout, float eps,
                                float base, uint32_t norm_group, float* qsrc, const WT* __restrict__ qw, uint32_t q_heads, uint32_t temp_every, float temp_coef,
-                               uint32_t hrot, const float* __restrict__ freqs, uint32_t horder, float* __restrict__ pooled, uint32_t pool, uint32_t pool_rows) {
+                               uint32_t hrot, const float* __restrict__ freqs, uint32_t horder, float* __restrict__ pooled, uint32_t pool, uint32_t pool_rows,
+                               float mag, uint32_t q_hs, float* qdst, uint32_t qdst_hs, uint32_t qdst_rs) {
     pdl_enter();
     if (pooled && blockIdx.x) {       // single-token steps: further CTAs average the block that ended just before this token
         pool_block(pooled, cache, ctl, 1u, cols, width, R, pool, pool_rows, 0u, (blockIdx.x - 1) * blockDim.x + threadIdx.x, (gridDim.x - 1) * blockDim.x);
         return;
     }
     __shared__ float sh[32];
-    extern __shared__ float cs_sn[];                   // head rotary: cosine | sine of the token's hrot / 2 angles, shared by all heads
+    extern __shared__ float cs_sn[];                   // rotary: cosine | sine of the token's angles (times the magnitude), shared by all heads
     const uint32_t t = blockIdx.x;
     const uint32_t pos = (uint32_t)ctl_word(ctl, ZG_CTL_POS) + t, slot = (uint32_t)ctl_word(ctl, ZG_CTL_SLOT);
     float* row = cache + ((size_t)slot * R + pos % R) * width;
@@ -114,7 +116,7 @@ __global__ void k_cache_append(float* __restrict__ cache, const float* __restric
         for (uint32_t i = threadIdx.x; i < hh; i += blockDim.x) {
             float sn, cs;
             if (freqs) sincosf((float)pos * freqs[i], &sn, &cs); else rotary_angle(pos, i, hrot, base, sn, cs);
-            cs_sn[i] = cs; cs_sn[hh + i] = sn;
+            cs_sn[i] = mag * cs; cs_sn[hh + i] = mag * sn;
         }
         __syncthreads();
         const uint32_t warp = threadIdx.x >> 5, lane = threadIdx.x & 31, nw = blockDim.x >> 5;
@@ -167,11 +169,25 @@ __global__ void k_cache_append(float* __restrict__ cache, const float* __restric
     const uint32_t half = rot / 2;
     for (uint32_t i = threadIdx.x; i < half; i += blockDim.x) {
         float sn, cs;
-        rotary_angle(pos, i, rot, base, sn, cs);
+        if (freqs) sincosf((float)pos * freqs[i], &sn, &cs); else rotary_angle(pos, i, rot, base, sn, cs);
+        sn *= mag; cs *= mag;
+        if (q_hs) { cs_sn[i] = cs; cs_sn[half + i] = sn; }
         const uint32_t a = normed + (layout == 0 ? 2 * i : i), b = normed + (layout == 0 ? 2 * i + 1 : i + half);
         const float u = s[a], w = s[b];
         row[a] = u * cs - w * sn;
         row[b] = w * cs + u * sn;
+    }
+    if (q_hs) {        // the rotated part of every query head, by the same angles: in place, or into the rows another op attends with
+        __syncthreads();
+        const float* q0 = qsrc + (size_t)t * src_rs;
+        float* d0 = qdst + (size_t)t * qdst_rs;
+        for (uint32_t e = threadIdx.x; e < q_heads * half; e += blockDim.x) {
+            const uint32_t hd = e / half, i = e % half, a = layout == 0 ? 2 * i : i, b = layout == 0 ? 2 * i + 1 : i + half;
+            const float u = q0[(size_t)hd * q_hs + a], w = q0[(size_t)hd * q_hs + b], cs = cs_sn[i], sn = cs_sn[half + i];
+            d0[(size_t)hd * qdst_hs + a] = u * cs - w * sn;
+            d0[(size_t)hd * qdst_hs + b] = w * cs + u * sn;
+        }
+        q_heads = 0;
     }
     for (uint32_t c = normed + rot + threadIdx.x; c < cols; c += blockDim.x) row[c] = s[c];
     if (q_heads) {     // the step's QUERY heads are normed in place by the same launch (per head, one shared weight), times a temperature that grows with the position
@@ -793,8 +809,11 @@ __global__ void k_gate(float* __restrict__ dst, const float* __restrict__ gate, 
 struct HlArgs {
     float* dst; const float* src; const float* gate;   // gate: output (h, n) of row m is multiplied by sigmoid(gate[m, (h N + n) / group])
     uint32_t T, H, N, K, src_hs, src_rs, dst_hs, dst_rs, gate_rs, gate_group;
+    uint32_t n_last, act; float act_p;      // outputs of the last head and the activation they alone pass
 };
+__device__ __forceinline__ uint32_t hl_outputs(const HlArgs& a, uint32_t h) { return h + 1 == a.H ? a.n_last : a.N; }
 __device__ __forceinline__ float hl_gated(const HlArgs& a, float v, uint32_t m, uint32_t h, uint32_t n) {
+    if (a.act && h + 1 == a.H) v = seq_epilogue(v, a.act, a.act_p);
     return a.gate ? v * sigmoidf_(a.gate[(size_t)m * a.gate_rs + (h * a.N + n) / a.gate_group]) : v;
 }
 constexpr int kHlRows = 8;
@@ -804,7 +823,7 @@ template <typename WT, bool VEC>
 __global__ void k_head_linear_rows(HlArgs a, const WT* __restrict__ W) {
     pdl_enter();
     const uint32_t n = blockIdx.x * (blockDim.x >> 5) + (threadIdx.x >> 5), lane = threadIdx.x & 31, h = blockIdx.y;
-    if (n >= a.N) return;
+    if (n >= hl_outputs(a, h)) return;
     const WT* w = W + ((size_t)h * a.N + n) * a.K;
     const float* x = a.src + (size_t)h * a.src_hs;
     float acc[kHlRows];
@@ -843,13 +862,69 @@ __global__ void k_head_linear_rows(HlArgs a, const WT* __restrict__ W) {
         }
     }
 }
+// Wide heads, few rows (every head a whole matrix product, as the stacked projections of a token-mixing layer): as the LINEAR op's row
+// kernel, the input row is staged once per CTA, the weight row is pulled toward L2 before the wait on the predecessor, and four
+// weight vectors per lane are in flight.
+template <typename WT, int MR>
+__global__ void k_head_linear_wide(HlArgs a, const WT* __restrict__ W) {
+    asm volatile("griddepcontrol.launch_dependents;" ::: "memory");
+    constexpr int V = WVec<WT>::n;
+    const uint32_t n = blockIdx.x * (blockDim.x >> 5) + (threadIdx.x >> 5), lane = threadIdx.x & 31, h = blockIdx.y, N = hl_outputs(a, h);
+    if (blockIdx.x * (blockDim.x >> 5) >= N) return;
+    const WT* w = W + ((size_t)h * a.N + n) * a.K;
+    if (n < N)
+        for (size_t b = (size_t)lane * 128; b < (size_t)a.K * sizeof(WT); b += 32 * 128) asm volatile("prefetch.global.L2 [%0];" ::"l"(reinterpret_cast<const char*>(w) + b));
+    asm volatile("griddepcontrol.wait;" ::: "memory");
+    extern __shared__ __align__(16) float xs[];        // [T][K]
+    const float* x = a.src + (size_t)h * a.src_hs;
+    for (uint32_t e = threadIdx.x; e < a.T * (a.K / 4); e += blockDim.x)
+        reinterpret_cast<float4*>(xs)[e] = *reinterpret_cast<const float4*>(x + (size_t)(e / (a.K / 4)) * a.src_rs + 4 * (e % (a.K / 4)));
+    __syncthreads();
+    if (n >= N) return;
+    float acc[MR];
+#pragma unroll
+    for (int m = 0; m < MR; m++) acc[m] = 0.0f;
+    auto fma_vec = [&](const float* wv, uint32_t k) {
+#pragma unroll
+        for (int m = 0; m < MR; m++) {
+            if (m < (int)a.T) {
+                const float4* xv = reinterpret_cast<const float4*>(xs + (size_t)m * a.K + k);
+#pragma unroll
+                for (int i = 0; i < V / 4; i++) {
+                    const float4 q = xv[i];
+                    acc[m] = fmaf(q.x, wv[4 * i], fmaf(q.y, wv[4 * i + 1], fmaf(q.z, wv[4 * i + 2], fmaf(q.w, wv[4 * i + 3], acc[m]))));
+                }
+            }
+        }
+    };
+    uint32_t k = lane * V;
+    for (; k + 96 * V < a.K; k += 128 * V) {
+        float w0[V], w1[V], w2[V], w3[V];
+        wld_vec<WT>(w + k, w0); wld_vec<WT>(w + k + 32 * V, w1); wld_vec<WT>(w + k + 64 * V, w2); wld_vec<WT>(w + k + 96 * V, w3);
+        fma_vec(w0, k); fma_vec(w1, k + 32 * V); fma_vec(w2, k + 64 * V); fma_vec(w3, k + 96 * V);
+    }
+    for (; k < a.K; k += 32 * V) {
+        float w0[V];
+        wld_vec<WT>(w + k, w0);
+        fma_vec(w0, k);
+    }
+#pragma unroll
+    for (int m = 0; m < MR; m++) {
+        if (m < (int)a.T) {
+            const float s = warp_sum(acc[m]);
+            if (lane == 0) a.dst[(size_t)m * a.dst_rs + (size_t)h * a.dst_hs + n] = hl_gated(a, s, m, h, n);
+        }
+    }
+}
+constexpr uint32_t kHlWideK = 256;     // from this many inputs per head on
 // many rows, exact f32: 64 x 64 tile of one head, 16-deep k slices, 4 x 4 outputs per thread
 constexpr int kHlTM = 64, kHlTN = 64, kHlTK = 16;
 template <typename WT>
 __global__ void __launch_bounds__(256) k_head_linear_tile(HlArgs a, const WT* __restrict__ W) {
     __shared__ float As[kHlTK][kHlTM + 4];
     __shared__ float Ws[kHlTK][kHlTN + 4];
-    const uint32_t h = blockIdx.z, m0 = blockIdx.y * kHlTM, n0 = blockIdx.x * kHlTN;
+    const uint32_t h = blockIdx.z, m0 = blockIdx.y * kHlTM, n0 = blockIdx.x * kHlTN, N = hl_outputs(a, h);
+    if (n0 >= N) return;
     const uint32_t tx = threadIdx.x & 15, ty = threadIdx.x >> 4;
     const float* src = a.src + (size_t)h * a.src_hs;
     const WT* Wh = W + (size_t)h * a.N * a.K;
@@ -859,7 +934,7 @@ __global__ void __launch_bounds__(256) k_head_linear_tile(HlArgs a, const WT* __
             const uint32_t r = e / kHlTK, kk = e % kHlTK;
             const uint32_t m = m0 + r, k = k0 + kk, n = n0 + r;
             As[kk][r] = (m < a.T && k < a.K) ? src[(size_t)m * a.src_rs + k] : 0.0f;
-            Ws[kk][r] = (n < a.N && k < a.K) ? wld(Wh, (size_t)n * a.K + k) : 0.0f;
+            Ws[kk][r] = (n < N && k < a.K) ? wld(Wh, (size_t)n * a.K + k) : 0.0f;
         }
         __syncthreads();
 #pragma unroll
@@ -881,7 +956,7 @@ __global__ void __launch_bounds__(256) k_head_linear_tile(HlArgs a, const WT* __
 #pragma unroll
         for (int j = 0; j < 4; j++) {
             const uint32_t n = n0 + tx * 4 + j;
-            if (n < a.N) a.dst[(size_t)m * a.dst_rs + (size_t)h * a.dst_hs + n] = hl_gated(a, acc[i][j], m, h, n);
+            if (n < N) a.dst[(size_t)m * a.dst_rs + (size_t)h * a.dst_hs + n] = hl_gated(a, acc[i][j], m, h, n);
         }
     }
 }
@@ -955,12 +1030,19 @@ bool zg_mix_op_valid(const ZgOp& op, const size_t* elems, size_t n_bufs, char* w
             const bool turn_only = s.n[13] == 2;
             if (s.n[13] > 2 || (s.n[13] && !s.n[10])) return fail("cache_append: order of norm and rotation");
             if (normed && !turn_only && !wfits(3, s.n[7], s.off[2], s.n[9] ? s.n[9] : normed)) return fail("cache_append: norm weight");
-            if (rot && !(s.f[1] > 0.0f)) return fail("cache_append: rotary base");
+            if (rot && (s.buf[4] != ZG_NO_BUF ? !fits(4, s.off[7], rot / 2) : !(s.f[1] > 0.0f))) return fail("cache_append: rotary frequencies");
+            if (s.f[3] < 0.0f) return fail("cache_append: rotary magnitude");
+            if (s.n[14]) {     // the rotated part of the query heads
+                const size_t qh = s.off[5], hs = s.n[14], dhs = s.n[15], end = s.off[3] + (qh - 1) * hs + rot;
+                if (!rot || !qh || s.n[9] || hs < rot || end > srs || !fits(1, 0, (T - 1) * srs + end)) return fail("cache_append: rotated query heads");
+                if (s.off[3] < s.off[0] + cols && s.off[0] < end) return fail("cache_append: query heads overlap the appended columns");
+                if (s.buf[6] != ZG_NO_BUF && (dhs < s.off[4] + rot || !fits(6, 0, T * qh * dhs) || s.buf[6] == s.buf[1] || s.buf[6] == s.buf[0])) return fail("cache_append: destination of the query heads");
+            }
             if (s.n[10]) {     // rotary inside every normed head, before its norm
                 if (!normed || !s.n[9] || rot || s.n[10] % 2 || s.n[10] > s.n[9]) return fail("cache_append: head rotary");
                 if (s.buf[4] != ZG_NO_BUF ? !fits(4, s.off[7], s.n[10] / 2) : !(s.f[1] > 0.0f)) return fail("cache_append: head rotary frequencies");
             }
-            if (s.off[5]) {    // query heads normed in place in the source rows
+            if (s.off[5] && !s.n[14]) {    // query heads normed in place in the source rows
                 const size_t qh = s.off[5], hd = s.n[9];
                 if (!normed || !hd || s.off[3] + qh * hd > srs || !fits(1, 0, (T - 1) * srs + s.off[3] + qh * hd) || (!turn_only && !wfits(3, s.n[7], s.off[4], hd))) return fail("cache_append: query heads");
                 if (s.off[3] < s.off[0] + cols && s.off[0] < s.off[3] + qh * hd) return fail("cache_append: query heads overlap the appended columns");
@@ -1008,10 +1090,12 @@ bool zg_mix_op_valid(const ZgOp& op, const size_t* elems, size_t n_bufs, char* w
             return true;
         }
         case ZG_OP_HEAD_LINEAR: {
-            const size_t T = s.n[0], H = s.n[1], N = s.n[2], K = s.n[3], shs = s.n[4], srs = s.n[5], dhs = s.n[6], drs = s.n[7];
-            if (!T || !H || !N || !K || shs < K || dhs < N || s.off[1] + (H - 1) * shs + K > srs || s.off[2] + (H - 1) * dhs + N > drs) return fail("head_linear: shape");
-            if (!fits(0, 0, (T - 1) * drs + s.off[2] + (H - 1) * dhs + N) || !fits(1, 0, (T - 1) * srs + s.off[1] + (H - 1) * shs + K) || !wfits(2, s.n[8], s.off[0], H * N * K))
+            const size_t T = s.n[0], H = s.n[1], N = s.n[2], K = s.n[3], shs = s.n[4], srs = s.n[5], dhs = s.n[6], drs = s.n[7], last = s.n[10] ? s.n[10] : N;
+            if (!T || !H || !N || !K || shs < K || dhs < N || s.off[1] + (H - 1) * shs + K > srs || s.off[2] + (H - 1) * dhs + last > drs) return fail("head_linear: shape");
+            if (!fits(0, 0, (T - 1) * drs + s.off[2] + (H - 1) * dhs + last) || !fits(1, 0, (T - 1) * srs + s.off[1] + (H - 1) * shs + K) || !wfits(2, s.n[8], s.off[0], ((H - 1) * N + last) * K))
                 return fail("head_linear: extent");
+            if (s.n[11] > 6 || (s.n[11] == 5 && !(s.f[0] > 0.0f)) || s.n[12] > 1) return fail("head_linear: activation or precision");
+            if (s.buf[3] != ZG_NO_BUF && (s.n[10] || s.n[11] || s.n[12])) return fail("head_linear: a gate goes with equal heads, no activation and exact products");
             if (s.buf[0] == s.buf[1]) return fail("head_linear: in place");
             if (s.buf[3] != ZG_NO_BUF) {
                 const size_t group = s.n[9], grs = s.off[4];
@@ -1030,11 +1114,18 @@ bool zg_mix_op_valid(const ZgOp& op, const size_t* elems, size_t n_bufs, char* w
 }
 
 uint32_t zg_mix_op_writes(uint32_t tag) {
-    if (tag == ZG_OP_CACHE_APPEND) return 1u | (1u << 1) | (1u << 5);   // the source rows too: query heads may be normed in place; pooled blocks, where named
+    if (tag == ZG_OP_CACHE_APPEND) return 1u | (1u << 1) | (1u << 5) | (1u << 6);   // the source rows too: query heads may be normed or turned in place; pooled blocks and turned query heads, where named
     return tag == ZG_OP_TOKEN_SHIFT ? (1u | (1u << 3)) : 1u;
 }
 
+// HEAD_LINEAR whose inputs may be rounded (n12) runs many rows on the tensor cores, as LINEAR does
+static bool hl_tensor(const ZgSeqOp& s) {
+    static const bool enabled = [] { const char* e = getenv("ZG_DENSE_GEMM"); return !(e && e[0] == '0'); }();
+    return enabled && s.n[12] && s.n[8] == ZG_W_BF16 && zg_dense_gemm_batched_usable(s.n[0], s.n[2], s.n[3], s.n[11]);
+}
+
 size_t zg_mix_op_scratch_elems(const ZgOp& op) {
+    if (op.tag == ZG_OP_HEAD_LINEAR) return hl_tensor(op.u.seq) ? zg_dense_gemm_batched_scratch_elems(op.u.seq.n[1], op.u.seq.n[0], op.u.seq.n[3]) : 0;
     if (op.tag != ZG_OP_CACHED_ATTENTION) return 0;
     const ZgSeqOp& s = op.u.seq;
     const uint32_t S = ca_splits(s);
@@ -1068,11 +1159,13 @@ bool zg_launch_mix_op(const ZgOp& op, float* const* bufs, float* scratch, cudaSt
         case ZG_OP_CACHE_APPEND: {
             float* pooled = s.n[11] ? bufs[s.buf[5]] + s.off[1] : nullptr;
             const bool turn_only = s.n[13] == 2;
-            ZG_SEQ_WDT(s.n[5] ? s.n[7] : ZG_W_F32, launch_pdl(k_cache_append<WT>, dim3(s.n[0] + (pooled && s.n[0] == 1 ? (s.n[1] + 255) / 256 : 0)), dim3(s.off[5] ? 256 : 128), (size_t)s.n[10] * sizeof(float), st, bufs[s.buf[0]] + s.off[1], bufs[s.buf[1]] + s.off[0], bufs[s.buf[2]],
+            ZG_SEQ_WDT(s.n[5] ? s.n[7] : ZG_W_F32, launch_pdl(k_cache_append<WT>, dim3(s.n[0] + (pooled && s.n[0] == 1 ? (s.n[1] + 255) / 256 : 0)), dim3(s.off[5] ? 256 : 128), (size_t)(s.n[10] ? s.n[10] : s.n[14] ? s.n[6] : 0) * sizeof(float), st, bufs[s.buf[0]] + s.off[1], bufs[s.buf[1]] + s.off[0], bufs[s.buf[2]],
                                                              s.n[5] && !turn_only ? wptr<WT>(bufs, s.buf[3], s.off[2]) : nullptr, s.n[1], s.n[2], s.n[3], s.n[4], s.n[5], s.n[6], s.n[8], s.f[0], s.f[1], s.n[9],
-                                                             s.off[5] ? bufs[s.buf[1]] + s.off[3] : nullptr, s.off[5] && !turn_only ? wptr<WT>(bufs, s.buf[3], s.off[4]) : nullptr, s.off[5], s.off[6], s.f[2],
-                                                             s.n[10], s.n[10] && s.buf[4] != ZG_NO_BUF ? (const float*)(bufs[s.buf[4]] + s.off[7]) : (const float*)nullptr, s.n[13],
-                                                             s.n[0] == 1 ? pooled : (float*)nullptr, s.n[11], s.n[12]));
+                                                             s.off[5] ? bufs[s.buf[1]] + s.off[3] : nullptr, s.off[5] && !turn_only && !s.n[14] ? wptr<WT>(bufs, s.buf[3], s.off[4]) : nullptr, s.off[5], s.off[6], s.f[2],
+                                                             s.n[10], (s.n[10] || s.n[6]) && s.buf[4] != ZG_NO_BUF ? (const float*)(bufs[s.buf[4]] + s.off[7]) : (const float*)nullptr, s.n[13],
+                                                             s.n[0] == 1 ? pooled : (float*)nullptr, s.n[11], s.n[12], s.f[3] > 0.0f ? s.f[3] : 1.0f, s.n[14],
+                                                             s.n[14] ? (s.buf[6] != ZG_NO_BUF ? bufs[s.buf[6]] + s.off[4] : bufs[s.buf[1]] + s.off[3]) : (float*)nullptr,
+                                                             s.buf[6] != ZG_NO_BUF ? s.n[15] : s.n[14], s.buf[6] != ZG_NO_BUF ? s.off[5] * s.n[15] : s.n[2]));
             ZG_SEQ_CHECK();
             if (pooled && s.n[0] > 1) {
                 launch_pdl(k_block_pool, dim3((s.n[0] - 1) / s.n[11] + 1, (s.n[1] + 127) / 128), dim3(128), 0, st, pooled, (const float*)(bufs[s.buf[0]] + s.off[1]), (const float*)bufs[s.buf[2]],
@@ -1154,13 +1247,21 @@ bool zg_launch_mix_op(const ZgOp& op, float* const* bufs, float* scratch, cudaSt
             a.dst = bufs[s.buf[0]] + s.off[2]; a.src = bufs[s.buf[1]] + s.off[1];
             a.T = s.n[0]; a.H = s.n[1]; a.N = s.n[2]; a.K = s.n[3]; a.src_hs = s.n[4]; a.src_rs = s.n[5]; a.dst_hs = s.n[6]; a.dst_rs = s.n[7];
             a.gate = s.buf[3] != ZG_NO_BUF ? bufs[s.buf[3]] + s.off[3] : nullptr; a.gate_rs = s.off[4]; a.gate_group = s.n[9];
+            a.n_last = s.n[10] ? s.n[10] : a.N; a.act = s.n[11]; a.act_p = s.f[0];
+            const uint32_t widest = a.n_last > a.N ? a.n_last : a.N;
+            if (scratch && hl_tensor(s) && (reinterpret_cast<uintptr_t>(wptr<bf16>(bufs, s.buf[2], s.off[0])) & 15) == 0)
+                return zg_dense_gemm_batched_launch(wptr<bf16>(bufs, s.buf[2], s.off[0]), a.src, a.dst, a.H, a.T, a.N, a.n_last, a.K, a.src_hs, a.src_rs, a.dst_hs, a.dst_rs, scratch, st, a.act, a.act_p);
             ZG_SEQ_WDT(s.n[8], {
                 const WT* W = wptr<WT>(bufs, s.buf[2], s.off[0]);
                 constexpr uint32_t V = WVec<WT>::n;
                 const bool vec = a.K % V == 0 && a.src_hs % 4 == 0 && a.src_rs % 4 == 0 && ((reinterpret_cast<uintptr_t>(W) | reinterpret_cast<uintptr_t>(a.src)) & 15) == 0;
-                if (a.T <= (uint32_t)kHlRows && vec) launch_pdl(k_head_linear_rows<WT, true>, dim3((a.N + 7) / 8, a.H), dim3(256), 0, st, a, W);
-                else if (a.T <= (uint32_t)kHlRows) launch_pdl(k_head_linear_rows<WT, false>, dim3((a.N + 7) / 8, a.H), dim3(256), 0, st, a, W);
-                else k_head_linear_tile<WT><<<dim3((a.N + kHlTN - 1) / kHlTN, (a.T + kHlTM - 1) / kHlTM, a.H), 256, 0, st>>>(a, W);
+                const size_t xs_bytes = (size_t)a.T * a.K * sizeof(float);
+                const bool wide = vec && a.K >= kHlWideK && xs_bytes <= 48 * 1024;
+                if (a.T == 1 && wide) launch_pdl(k_head_linear_wide<WT, 1>, dim3((widest + 7) / 8, a.H), dim3(256), xs_bytes, st, a, W);
+                else if (a.T <= (uint32_t)kHlRows && wide) launch_pdl(k_head_linear_wide<WT, kHlRows>, dim3((widest + 7) / 8, a.H), dim3(256), xs_bytes, st, a, W);
+                else if (a.T <= (uint32_t)kHlRows && vec) launch_pdl(k_head_linear_rows<WT, true>, dim3((widest + 7) / 8, a.H), dim3(256), 0, st, a, W);
+                else if (a.T <= (uint32_t)kHlRows) launch_pdl(k_head_linear_rows<WT, false>, dim3((widest + 7) / 8, a.H), dim3(256), 0, st, a, W);
+                else k_head_linear_tile<WT><<<dim3((widest + kHlTN - 1) / kHlTN, (a.T + kHlTM - 1) / kHlTM, a.H), 256, 0, st>>>(a, W);
             });
             ZG_SEQ_CHECK();
             return true;

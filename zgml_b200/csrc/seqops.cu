@@ -15,7 +15,7 @@ namespace {
 // ── EMBED ─────────────────────────────────────────────────────────────────────────────────────────────────────────
 template <typename WT>
 __global__ void k_embed(float* __restrict__ dst, const float* __restrict__ ctl, const WT* __restrict__ table, uint32_t D, float scale,
-                        const WT* __restrict__ positions, const WT* __restrict__ bigram, uint32_t buckets, uint32_t mul_prev, uint32_t mul_cur) {
+                        const WT* __restrict__ positions, const WT* __restrict__ bigram, uint32_t buckets, uint32_t mul_prev, uint32_t mul_cur, const WT* __restrict__ dyt) {
     pdl_enter();
     const uint32_t t = blockIdx.x, c = blockIdx.y * blockDim.x + threadIdx.x;
     if (c >= D) return;
@@ -28,12 +28,15 @@ __global__ void k_embed(float* __restrict__ dst, const float* __restrict__ ctl, 
     } else if (positions) {       // a learned position row, not scaled
         add = wld(positions, ((size_t)ctl_word(ctl, ZG_CTL_POS) + t) * D + c);
     }
-    dst[(size_t)t * D + c] = fmaf(wld(table, (size_t)id * D + c), scale, add);
+    float x = fmaf(wld(table, (size_t)id * D + c), scale, add);
+    if (dyt) x = fmaf(tanhf(wld(dyt, (size_t)2 * D) * x), wld(dyt, c), wld(dyt, (size_t)D + c));      // Dynamic Tanh: weight | bias | alpha
+    dst[(size_t)t * D + c] = x;
 }
 
 // ── LINEAR, few rows (decode): one warp per output feature, the weight row streamed once for all rows ─────────────────
 constexpr int kGemvRows = 8;
-template <typename WT>
+// PAIRS: weight rows 2n and 2n + 1 are a gate and what it multiplies, dst[., n] = act(row 2n . x) * (row 2n + 1 . x)
+template <typename WT, bool PAIRS>
 __global__ void k_linear_rows(float* __restrict__ dst, const float* __restrict__ src, const WT* __restrict__ W, const WT* __restrict__ bias,
                               uint32_t M, uint32_t N, uint32_t K, uint32_t src_rs, uint32_t dst_rs, SeqAct act, const float* __restrict__ ctl,
                               uint32_t slot_stride) {
@@ -41,28 +44,32 @@ __global__ void k_linear_rows(float* __restrict__ dst, const float* __restrict__
     if (ctl) src += (size_t)ctl_word(ctl, ZG_CTL_SLOT) * slot_stride;      // the rows of a per-sequence state buffer
     const uint32_t n = blockIdx.x * (blockDim.x >> 5) + (threadIdx.x >> 5), lane = threadIdx.x & 31;
     if (n >= N) return;
-    const WT* w = W + (size_t)n * K;
-    float acc[kGemvRows];
+    const WT* w = W + (size_t)(PAIRS ? 2 * n : n) * K;
+    float acc[kGemvRows], up[kGemvRows];
 #pragma unroll
-    for (int m = 0; m < kGemvRows; m++) acc[m] = 0.0f;
+    for (int m = 0; m < kGemvRows; m++) acc[m] = up[m] = 0.0f;
     for (uint32_t k = lane; k < K; k += 32) {
-        const float wv = wld(w, k);
+        const float wv = wld(w, k), uv = PAIRS ? wld(w, (size_t)K + k) : 0.0f;
 #pragma unroll
         for (int m = 0; m < kGemvRows; m++)
-            if (m < (int)M) acc[m] = fmaf(src[(size_t)m * src_rs + k], wv, acc[m]);
+            if (m < (int)M) {
+                const float x = src[(size_t)m * src_rs + k];
+                acc[m] = fmaf(x, wv, acc[m]);
+                if (PAIRS) up[m] = fmaf(x, uv, up[m]);
+            }
     }
-    const float b = bias ? wld(bias, n) : 0.0f;
+    const float b = bias && !PAIRS ? wld(bias, n) : 0.0f;
 #pragma unroll
     for (int m = 0; m < kGemvRows; m++) {
         if (m < (int)M) {
-            const float s = warp_sum(acc[m]);
-            if (lane == 0) dst[(size_t)m * dst_rs + n] = seq_epilogue(s + b, act, n);
+            const float s = warp_sum(acc[m]), u = PAIRS ? warp_sum(up[m]) : 1.0f;
+            if (lane == 0) dst[(size_t)m * dst_rs + n] = PAIRS ? seq_epilogue(s, act.kind, act.p) * u : seq_epilogue(s + b, act, n);
         }
     }
 }
 // The activation rows are staged once per CTA in shared memory (float4 reads, no per-weight global loads); four weight
 // vectors per lane are in flight per trip.
-template <typename WT, int MR>
+template <typename WT, int MR, bool PAIRS>
 __global__ void k_linear_rows_vec(float* __restrict__ dst, const float* __restrict__ src, const WT* __restrict__ W, const WT* __restrict__ bias,
                                   uint32_t M, uint32_t N, uint32_t K, uint32_t src_rs, uint32_t dst_rs, SeqAct act, const float* __restrict__ ctl,
                                   uint32_t slot_stride) {
@@ -72,8 +79,8 @@ __global__ void k_linear_rows_vec(float* __restrict__ dst, const float* __restri
     {
         const uint32_t n0 = blockIdx.x * (blockDim.x >> 5) + (threadIdx.x >> 5);
         if (n0 < N) {
-            const char* wb = reinterpret_cast<const char*>(W + (size_t)n0 * K);
-            for (size_t b = (size_t)(threadIdx.x & 31) * 128; b < (size_t)K * sizeof(WT); b += 32 * 128)
+            const char* wb = reinterpret_cast<const char*>(W + (size_t)(PAIRS ? 2 * n0 : n0) * K);
+            for (size_t b = (size_t)(threadIdx.x & 31) * 128; b < (size_t)(PAIRS ? 2 : 1) * K * sizeof(WT); b += 32 * 128)
                 asm volatile("prefetch.global.L2 [%0];" ::"l"(wb + b));
         }
     }
@@ -85,11 +92,11 @@ __global__ void k_linear_rows_vec(float* __restrict__ dst, const float* __restri
     __syncthreads();
     const uint32_t n = blockIdx.x * (blockDim.x >> 5) + (threadIdx.x >> 5), lane = threadIdx.x & 31;
     if (n >= N) return;
-    const WT* w = W + (size_t)n * K;
-    float acc[MR];
+    const WT* w = W + (size_t)(PAIRS ? 2 * n : n) * K;
+    float acc[MR], up[MR];
 #pragma unroll
-    for (int m = 0; m < MR; m++) acc[m] = 0.0f;
-    auto fma_vec = [&](const float* wv, uint32_t k) {
+    for (int m = 0; m < MR; m++) acc[m] = up[m] = 0.0f;
+    auto fma_into = [&](float (&sum)[MR], const float* wv, uint32_t k) {
 #pragma unroll
         for (int m = 0; m < MR; m++) {
             if (m < (int)M) {
@@ -97,53 +104,83 @@ __global__ void k_linear_rows_vec(float* __restrict__ dst, const float* __restri
 #pragma unroll
                 for (int i = 0; i < V / 4; i++) {
                     const float4 xv = x[i];
-                    acc[m] = fmaf(xv.x, wv[4 * i], fmaf(xv.y, wv[4 * i + 1], fmaf(xv.z, wv[4 * i + 2], fmaf(xv.w, wv[4 * i + 3], acc[m]))));
+                    sum[m] = fmaf(xv.x, wv[4 * i], fmaf(xv.y, wv[4 * i + 1], fmaf(xv.z, wv[4 * i + 2], fmaf(xv.w, wv[4 * i + 3], sum[m]))));
                 }
             }
         }
     };
+    auto fma_vec = [&](const float* wv, uint32_t k) { fma_into(acc, wv, k); };
     uint32_t k = lane * V;
-    for (; k + 96 * V < K; k += 128 * V) {
-        float w0[V], w1[V], w2[V], w3[V];
-        wld_vec<WT>(w + k, w0);
-        wld_vec<WT>(w + k + 32 * V, w1);
-        wld_vec<WT>(w + k + 64 * V, w2);
-        wld_vec<WT>(w + k + 96 * V, w3);
-        fma_vec(w0, k);
-        fma_vec(w1, k + 32 * V);
-        fma_vec(w2, k + 64 * V);
-        fma_vec(w3, k + 96 * V);
-    }
-    for (; k + 32 * V < K; k += 64 * V) {
-        float w0[V], w1[V];
-        wld_vec<WT>(w + k, w0);
-        wld_vec<WT>(w + k + 32 * V, w1);
-        fma_vec(w0, k);
-        fma_vec(w1, k + 32 * V);
-    }
-    if (k < K) {
-        float w0[V];
-        wld_vec<WT>(w + k, w0);
-        fma_vec(w0, k);
-    }
-    const float b = bias ? wld(bias, n) : 0.0f;
+    if constexpr (PAIRS) {                             // both rows' vectors in flight together
+        const WT* wu = w + K;
+        for (; k + 32 * V < K; k += 64 * V) {
+            float g0[V], g1[V], u0[V], u1[V];
+            wld_vec<WT>(w + k, g0);
+            wld_vec<WT>(wu + k, u0);
+            wld_vec<WT>(w + k + 32 * V, g1);
+            wld_vec<WT>(wu + k + 32 * V, u1);
+            fma_into(acc, g0, k); fma_into(up, u0, k);
+            fma_into(acc, g1, k + 32 * V); fma_into(up, u1, k + 32 * V);
+        }
+        if (k < K) {
+            float g0[V], u0[V];
+            wld_vec<WT>(w + k, g0);
+            wld_vec<WT>(wu + k, u0);
+            fma_into(acc, g0, k); fma_into(up, u0, k);
+        }
 #pragma unroll
-    for (int m = 0; m < MR; m++) {
-        if (m < (int)M) {
-            const float s = warp_sum(acc[m]);
-            if (lane == 0) dst[(size_t)m * dst_rs + n] = seq_epilogue(s + b, act, n);
+        for (int m = 0; m < MR; m++) {
+            if (m < (int)M) {
+                const float g = warp_sum(acc[m]), u = warp_sum(up[m]);
+                if (lane == 0) dst[(size_t)m * dst_rs + n] = seq_epilogue(g, act.kind, act.p) * u;
+            }
+        }
+    } else {
+        for (; k + 96 * V < K; k += 128 * V) {
+            float w0[V], w1[V], w2[V], w3[V];
+            wld_vec<WT>(w + k, w0);
+            wld_vec<WT>(w + k + 32 * V, w1);
+            wld_vec<WT>(w + k + 64 * V, w2);
+            wld_vec<WT>(w + k + 96 * V, w3);
+            fma_vec(w0, k);
+            fma_vec(w1, k + 32 * V);
+            fma_vec(w2, k + 64 * V);
+            fma_vec(w3, k + 96 * V);
+        }
+        for (; k + 32 * V < K; k += 64 * V) {
+            float w0[V], w1[V];
+            wld_vec<WT>(w + k, w0);
+            wld_vec<WT>(w + k + 32 * V, w1);
+            fma_vec(w0, k);
+            fma_vec(w1, k + 32 * V);
+        }
+        if (k < K) {
+            float w0[V];
+            wld_vec<WT>(w + k, w0);
+            fma_vec(w0, k);
+        }
+        const float b = bias ? wld(bias, n) : 0.0f;
+#pragma unroll
+        for (int m = 0; m < MR; m++) {
+            if (m < (int)M) {
+                const float s = warp_sum(acc[m]);
+                if (lane == 0) dst[(size_t)m * dst_rs + n] = seq_epilogue(s + b, act, n);
+            }
         }
     }
 }
 
 // ── LINEAR, many rows (prefill), exact f32: 64 x 64 tile, 16-deep k slices, 4 x 4 outputs per thread ──────────────────
 constexpr int kTM = 64, kTN = 64, kTK = 16;
-template <typename WT>
+// rows_from > 0: only the rows of positions the sequence holds after this step matter (rows < position + rows_from)
+// PAIRS: N counts weight rows, gate and up rows in turns; columns n and n + 1 make output n / 2
+template <typename WT, bool PAIRS>
 __global__ void __launch_bounds__(256) k_linear_tile(float* __restrict__ dst, const float* __restrict__ src, const WT* __restrict__ W,
                                                      const WT* __restrict__ bias, uint32_t M, uint32_t N, uint32_t K, uint32_t src_rs,
-                                                     uint32_t dst_rs, SeqAct act, const float* __restrict__ ctl, uint32_t slot_stride) {
+                                                     uint32_t dst_rs, SeqAct act, const float* __restrict__ ctl, uint32_t slot_stride, uint32_t rows_from) {
     __shared__ float As[kTK][kTM + 4];
     __shared__ float Ws[kTK][kTN + 4];
+    if (rows_from && blockIdx.y * kTM >= (uint32_t)ctl_word(ctl, ZG_CTL_POS) + rows_from) return;
     if (ctl) src += (size_t)ctl_word(ctl, ZG_CTL_SLOT) * slot_stride;
     const uint32_t m0 = blockIdx.y * kTM, n0 = blockIdx.x * kTN;
     const uint32_t tx = threadIdx.x & 15, ty = threadIdx.x >> 4;   // outputs: rows ty * 4 + i, columns tx * 4 + j
@@ -174,9 +211,11 @@ __global__ void __launch_bounds__(256) k_linear_tile(float* __restrict__ dst, co
         const uint32_t m = m0 + ty * 4 + i;
         if (m >= M) continue;
 #pragma unroll
-        for (int j = 0; j < 4; j++) {
+        for (int j = 0; j < 4; j += PAIRS ? 2 : 1) {
             const uint32_t n = n0 + tx * 4 + j;
-            if (n < N) dst[(size_t)m * dst_rs + n] = seq_epilogue(acc[i][j] + (bias ? wld(bias, n) : 0.0f), act, n);
+            if (n >= N) continue;
+            if (PAIRS) dst[(size_t)m * dst_rs + n / 2] = seq_epilogue(acc[i][j], act.kind, act.p) * acc[i][min(j + 1, 3)];
+            else dst[(size_t)m * dst_rs + n] = seq_epilogue(acc[i][j] + (bias ? wld(bias, n) : 0.0f), act, n);
         }
     }
 }
@@ -898,10 +937,13 @@ __global__ void k_conv_advance(float* __restrict__ state, const float* __restric
 constexpr int kDeltaRows = 16, kDeltaTile = 16, kDeltaThreads = 128;
 // forms of the rule (op parameter n10): plain accumulation without unit vectors and correction (gated linear attention), the
 // decay as a tempered sigmoid, a SiLU output gate, an output scale, one decay per head instead of one per key channel
-constexpr uint32_t kDeltaPlain = 1, kDeltaSigmoidDecay = 2, kDeltaSiluGate = 4, kDeltaOutScale = 8, kDeltaHeadDecay = 16;
+// a read-out before the token's write with the token itself joining through a bonus per key channel (RWKV's time mixing), the decay
+// as exp(-exp(z)), an output norm whose weight is one vector over all heads
+constexpr uint32_t kDeltaPlain = 1, kDeltaSigmoidDecay = 2, kDeltaSiluGate = 4, kDeltaOutScale = 8, kDeltaHeadDecay = 16, kDeltaBonus = 32, kDeltaExpDecay = 64, kDeltaWideNorm = 128;
 // decay of one key channel from its logit z (the bias is already added): exp(-exp(A) softplus(z)), or sigmoid(z)^(1 / tau) =
-// exp(-softplus(-z) / tau)
+// exp(-softplus(-z) / tau), or exp(-exp(z))
 __device__ __forceinline__ float delta_decay(float z, float Ah, uint32_t form, float inv_tau) {
+    if (form & kDeltaExpDecay) return expf(-expf(z));
     return (form & kDeltaSigmoidDecay) ? expf(-softplusf_(-z) * inv_tau) : expf(-Ah * softplusf_(z));
 }
 template <typename WT>
@@ -909,11 +951,12 @@ __global__ void __launch_bounds__(kDeltaThreads) k_delta_rule(
     float* __restrict__ dst, const float* __restrict__ qkv, const float* __restrict__ betab, const float* __restrict__ ab, const WT* __restrict__ wts,
     float* __restrict__ state, const float* __restrict__ ctl, uint32_t T, uint32_t H, uint32_t G, uint32_t dim, uint32_t vdim, uint32_t RS,
     uint32_t q_off, uint32_t k_off, uint32_t v_off, uint32_t beta_off, uint32_t A_off, uint32_t dt_off, uint32_t qkv_rs, uint32_t beta_rs,
-    uint32_t a_rs, float unit_eps, float q_scale, uint32_t form, float inv_tau, uint32_t dst_rs) {
+    uint32_t a_rs, float unit_eps, float q_scale, uint32_t form, float inv_tau, uint32_t dst_rs, uint32_t u_off) {
     pdl_enter();
     extern __shared__ float sm[];
     const bool plain = form & kDeltaPlain;             // no unit vectors, no correction: S <- g S + k v^T
     const bool head_decay = form & kDeltaHeadDecay;    // a row of `ab` holds one logit per head
+    const bool bonus = form & kDeltaBonus;             // plain: o = S^T q + (sum_i q_i u_i k_i) v before the write
     const uint32_t dpad = RS * kDeltaRows;             // rows incl. padding (k = q = 0, decay = 1 there)
     float* sk = sm;                                    // [tile][dpad]
     float* sq = sk + kDeltaTile * dpad;
@@ -931,7 +974,7 @@ __global__ void __launch_bounds__(kDeltaThreads) k_delta_rule(
         const uint32_t row = r * kDeltaRows + i;
         S[i] = (live && row < dim) ? S_g[(size_t)row * vdim + col] : 0.0f;
     }
-    const float Ah = (form & kDeltaSigmoidDecay) ? 0.0f : expf(wld(wts, (size_t)A_off + h));
+    const float Ah = (form & (kDeltaSigmoidDecay | kDeltaExpDecay)) ? 0.0f : expf(wld(wts, (size_t)A_off + h));
     const uint32_t warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
     for (uint32_t t0 = 0; t0 < T; t0 += kDeltaTile) {
         const uint32_t nt = min((uint32_t)kDeltaTile, T - t0);
@@ -955,7 +998,13 @@ __global__ void __launch_bounds__(kDeltaThreads) k_delta_rule(
                 sq[tt * dpad + c] = in ? qr[c] * qn : 0.0f;
                 sg[tt * dpad + c] = head_decay ? gh : in ? delta_decay(ar[c] + wld(wts, (size_t)dt_off + (size_t)h * dim + c), Ah, form, inv_tau) : 1.0f;
             }
-            if (lane == 0) sbeta[tt] = plain ? 1.0f : sigmoidf_(betab[(size_t)t * beta_rs + beta_off + h]);
+            float own = 1.0f;
+            if (bonus) {
+                own = 0.0f;
+                for (uint32_t c = lane; c < dim; c += 32) own = fmaf(qr[c] * qn * kr[c], wld(wts, (size_t)u_off + (size_t)h * dim + c), own);
+                own = warp_sum(own);
+            }
+            if (lane == 0) sbeta[tt] = plain ? own : sigmoidf_(betab[(size_t)t * beta_rs + beta_off + h]);
         }
         float vt[kDeltaTile];                              // the tile's values of this column: independent loads, issued together
 #pragma unroll
@@ -971,6 +1020,14 @@ __global__ void __launch_bounds__(kDeltaThreads) k_delta_rule(
             const float* q = sq + tt * dpad + r * kDeltaRows;
             const float* g = sg + tt * dpad + r * kDeltaRows;
             const float v = vt[tti];
+            if (bonus) {                                   // read first, then decay and write
+                float os = 0.0f;
+#pragma unroll
+                for (int i = 0; i < kDeltaRows; i++) { os = fmaf(S[i], q[i], os); S[i] = fmaf(S[i], g[i], k[i] * v); }
+                for (uint32_t o = 1; o < RS; o <<= 1) os += __shfl_xor_sync(0xffffffffu, os, o);
+                if (live && r == 0) dst[(size_t)t * dst_rs + (size_t)h * vdim + col] = fmaf(sbeta[tt], v, os);
+                continue;
+            }
             float ks = 0.0f;
 #pragma unroll
             for (int i = 0; i < kDeltaRows; i++) { S[i] *= g[i]; ks = fmaf(S[i], k[i], ks); }
@@ -1013,7 +1070,7 @@ template <typename WT>
 __global__ void k_delta_prepare(float* __restrict__ prep, const float* __restrict__ qkv, const float* __restrict__ betab, const float* __restrict__ ab,
                                 const WT* __restrict__ wts, uint32_t T, uint32_t H, uint32_t G, uint32_t dim, uint32_t dpad, uint32_t q_off,
                                 uint32_t k_off, uint32_t beta_off, uint32_t A_off, uint32_t dt_off, uint32_t qkv_rs, uint32_t beta_rs, uint32_t a_rs,
-                                float unit_eps, float q_scale, uint32_t form, float inv_tau) {
+                                float unit_eps, float q_scale, uint32_t form, float inv_tau, uint32_t u_off) {
     pdl_enter();
     const bool plain = form & kDeltaPlain, head_decay = form & kDeltaHeadDecay;
     const uint32_t w = blockIdx.x * (blockDim.x >> 5) + (threadIdx.x >> 5), lane = threadIdx.x & 31;
@@ -1023,10 +1080,11 @@ __global__ void k_delta_prepare(float* __restrict__ prep, const float* __restric
     const float* kr = qkv + (size_t)t * qkv_rs + k_off + (size_t)kv * dim;
     const float* ar = ab + (size_t)t * a_rs + (head_decay ? (size_t)h : (size_t)h * dim);
     float qq = 0.0f, kk = 0.0f, qk = 0.0f;
-    for (uint32_t c = lane; c < dim; c += 32) { const float a = qr[c], b = kr[c]; qq = fmaf(a, a, qq); kk = fmaf(b, b, kk); qk = fmaf(a, b, qk); }
+    for (uint32_t c = lane; c < dim; c += 32) { const float a = qr[c], b = kr[c]; qq = fmaf(a, a, qq); kk = fmaf(b, b, kk);
+        qk = fmaf(a, (form & kDeltaBonus) ? b * wld(wts, (size_t)u_off + (size_t)h * dim + c) : b, qk); }
     const float qn = plain ? q_scale : q_scale / sqrtf(warp_sum(qq) + unit_eps), kn = plain ? 1.0f : 1.0f / sqrtf(warp_sum(kk) + unit_eps);
     qk = warp_sum(qk) * qn * kn;
-    const float Ah = (form & kDeltaSigmoidDecay) ? 0.0f : expf(wld(wts, (size_t)A_off + h));
+    const float Ah = (form & (kDeltaSigmoidDecay | kDeltaExpDecay)) ? 0.0f : expf(wld(wts, (size_t)A_off + h));
     float* row = prep + ((size_t)h * T + t) * ((head_decay ? 2 : 3) * dpad + 4);
     const float gh = head_decay ? delta_decay(ar[0] + wld(wts, (size_t)dt_off + h), Ah, form, inv_tau) : 0.0f;
     for (uint32_t c = lane; c < dpad; c += 32) {
@@ -1043,7 +1101,8 @@ __device__ __forceinline__ void cp_async16(float* smem_dst, const float* gmem_sr
 // PLAIN: the accumulation without correction (u = v), which needs no product with k and only one reduction per token
 // HEADG: one decay per head and token.  It commutes with the sums over the key rows, so both dot products run on the state as
 // the token finds it and the decay joins the two results: u = beta (v - g S^T k), o = g S^T q + u (k . q), S <- g S + k u^T.
-template <uint32_t RS, bool PLAIN, bool HEADG>                     // row slices of a column: compile-time, so the shuffle steps unroll
+// BONUS (PLAIN): the state as the token finds it, not yet decayed, is what is read; k . q of the prepared row carries the bonus
+template <uint32_t RS, bool PLAIN, bool HEADG, bool BONUS>         // row slices of a column: compile-time, so the shuffle steps unroll
 __global__ void __launch_bounds__(kWalkThreads) k_delta_walk(float* __restrict__ dst, const float* __restrict__ qkv, const float* __restrict__ prep,
                                                                float* __restrict__ state, const float* __restrict__ ctl, uint32_t T, uint32_t H,
                                                                uint32_t dim, uint32_t vdim, uint32_t v_off, uint32_t qkv_rs, uint32_t dst_rs) {
@@ -1097,6 +1156,10 @@ __global__ void __launch_bounds__(kWalkThreads) k_delta_walk(float* __restrict__
                 const uint32_t at = (c * RS + r) * 4;
                 k4[c] = *reinterpret_cast<const float4*>(row + at);
                 const float4 q4 = *reinterpret_cast<const float4*>(row + dpad + at);
+                if (BONUS) {
+                    qs0 = fmaf(S[4 * c + 0], q4.x, qs0); qs1 = fmaf(S[4 * c + 1], q4.y, qs1);
+                    qs0 = fmaf(S[4 * c + 2], q4.z, qs0); qs1 = fmaf(S[4 * c + 3], q4.w, qs1);
+                }
                 if (!HEADG) {
                     g4[c] = *reinterpret_cast<const float4*>(row + 2 * dpad + at);
                     S[4 * c + 0] *= g4[c].x; S[4 * c + 1] *= g4[c].y; S[4 * c + 2] *= g4[c].z; S[4 * c + 3] *= g4[c].w;
@@ -1105,13 +1168,15 @@ __global__ void __launch_bounds__(kWalkThreads) k_delta_walk(float* __restrict__
                     ks0 = fmaf(S[4 * c + 0], k4[c].x, ks0); ks1 = fmaf(S[4 * c + 1], k4[c].y, ks1);
                     ks0 = fmaf(S[4 * c + 2], k4[c].z, ks0); ks1 = fmaf(S[4 * c + 3], k4[c].w, ks1);
                 }
-                qs0 = fmaf(S[4 * c + 0], q4.x, qs0); qs1 = fmaf(S[4 * c + 1], q4.y, qs1);
-                qs0 = fmaf(S[4 * c + 2], q4.z, qs0); qs1 = fmaf(S[4 * c + 3], q4.w, qs1);
+                if (!BONUS) {
+                    qs0 = fmaf(S[4 * c + 0], q4.x, qs0); qs1 = fmaf(S[4 * c + 1], q4.y, qs1);
+                    qs0 = fmaf(S[4 * c + 2], q4.z, qs0); qs1 = fmaf(S[4 * c + 3], q4.w, qs1);
+                }
             }
             float ks = ks0 + ks1, qs = qs0 + qs1;
 #pragma unroll
             for (uint32_t o = 1; o < RS; o <<= 1) { if (!PLAIN) ks += __shfl_xor_sync(0xffffffffu, ks, o); qs += __shfl_xor_sync(0xffffffffu, qs, o); }
-            if (HEADG) { ks *= gh; qs *= gh; }
+            if (HEADG) { ks *= gh; if (!BONUS) qs *= gh; }
             const float u = PLAIN ? v : beta * (v - ks);
 #pragma unroll
             for (int c = 0; c < kWalkRows / 4; c++) {
@@ -1144,7 +1209,7 @@ __global__ void __launch_bounds__(kWalkThreads) k_delta_walk(float* __restrict__
 // o / rms(o) * norm_w * sigmoid(gate) (or silu(gate)) * out_scale, one warp per (token, head), in place
 template <typename WT>
 __global__ void k_delta_out(float* __restrict__ dst, const float* __restrict__ gate, const WT* __restrict__ wts, uint32_t TH, uint32_t H,
-                            uint32_t vdim, uint32_t gate_rs, uint32_t nw_off, float eps, uint32_t dst_rs, uint32_t silu_gate, float out_scale) {
+                            uint32_t vdim, uint32_t gate_rs, uint32_t nw_off, float eps, uint32_t dst_rs, uint32_t silu_gate, float out_scale, uint32_t wide_norm) {
     pdl_enter();
     const uint32_t item = blockIdx.x * (blockDim.x >> 5) + (threadIdx.x >> 5), lane = threadIdx.x & 31;
     if (item >= TH) return;
@@ -1154,13 +1219,13 @@ __global__ void k_delta_out(float* __restrict__ dst, const float* __restrict__ g
     float q = 0.0f;
     for (uint32_t c = lane; c < vdim; c += 32) q = fmaf(o[c], o[c], q);
     const float inv = out_scale / sqrtf(warp_sum(q) / (float)vdim + eps);
-    for (uint32_t c = lane; c < vdim; c += 32) o[c] = o[c] * inv * wld(wts, (size_t)nw_off + c) * (silu_gate ? g[c] * sigmoidf_(g[c]) : sigmoidf_(g[c]));
+    for (uint32_t c = lane; c < vdim; c += 32) o[c] = o[c] * inv * wld(wts, (size_t)nw_off + (wide_norm ? (size_t)h * vdim : 0) + c) * (silu_gate ? g[c] * sigmoidf_(g[c]) : sigmoidf_(g[c]));
 }
 
 // ── ROUTE: one warp per token ────────────────────────────────────────────────────────────────────────────────────
 template <typename WT>
 __global__ void k_route(float* __restrict__ dst, const float* __restrict__ logits, const WT* __restrict__ corr, uint32_t T, uint32_t NE, uint32_t top,
-                        uint32_t logits_rs, uint32_t mode, uint32_t groups, uint32_t keep) {
+                        uint32_t logits_rs, uint32_t mode, uint32_t groups, uint32_t keep, float weight_scale) {
     pdl_enter();
     extern __shared__ float sm[];                      // [warps][NE + groups] choice scores, group scores
     const uint32_t warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
@@ -1224,6 +1289,7 @@ __global__ void k_route(float* __restrict__ dst, const float* __restrict__ logit
             reinterpret_cast<int*>(out)[0] = (int)bi;
             if (mode == 0) out[1] = bi < NE ? expf(z[bi] - mx) * inv : 0.0f;
             else if (mode == 2) { out[1] = bi < NE ? sigmoidf_(z[bi]) : 0.0f; chosen_sum += out[1]; }
+            else if (mode == 3) out[1] = bi < NE ? sigmoidf_(z[bi]) * weight_scale : 0.0f;
             else {
                 if (c == 0) first = best;
                 out[1] = bi < NE ? expf(best - first) : 0.0f;
@@ -1233,7 +1299,7 @@ __global__ void k_route(float* __restrict__ dst, const float* __restrict__ logit
         }
         __syncwarp();
     }
-    if (mode != 0 && lane == 0) {
+    if ((mode == 1 || mode == 2) && lane == 0) {
         const float norm = 1.0f / (mode == 2 ? chosen_sum + 1e-20f : chosen_sum);
         for (uint32_t c = 0; c < top; c++) dst[((size_t)t * top + c) * 2 + 1] *= norm;
     }
@@ -1474,6 +1540,7 @@ uint32_t zg_delta_row_slices(uint32_t dim) {
 
 // Static checks of a sequence op against the program's buffer sizes (f32 slots): shapes, strides and every extent.
 bool zg_seq_op_valid(const ZgOp& op, const size_t* elems, size_t n_bufs, char* why, size_t why_n) {
+    if (op.tag >= ZG_OP_STREAM_STEP) return zg_stream_op_valid(op, elems, n_bufs, why, why_n);
     if (op.tag >= ZG_OP_SSM_SCAN) return zg_rec_op_valid(op, elems, n_bufs, why, why_n);
     if (op.tag >= ZG_OP_TOKEN_SHIFT) return zg_mix_op_valid(op, elems, n_bufs, why, why_n);
     const ZgSeqOp& s = op.u.seq;
@@ -1489,12 +1556,15 @@ bool zg_seq_op_valid(const ZgOp& op, const size_t* elems, size_t n_bufs, char* w
             const size_t T = s.n[0], D = s.n[1];
             if (!fits(0, 0, T * D) || !fits(1, ZG_CTL_IDS, T) || !have(2)) return fail("embed: extent");
             if (s.n[4] && (s.n[3] || s.n[5] >= s.n[4] || s.n[6] >= s.n[4] || !wfits(2, s.off[2], ((size_t)s.n[4] + 1) * D))) return fail("embed: bigram table");
+            if (s.n[7] > 1 || (s.n[7] && !wfits(2, s.off[3], 2 * D + 1))) return fail("embed: norm");
             return true;
         }
         case ZG_OP_LINEAR: {
             const size_t M = s.n[0], N = s.n[1], K = s.n[2], srs = s.n[3], drs = s.n[4];
             if (!M || !N || !K || srs < K || drs < N) return fail("linear: shape");
-            if (!fits(0, s.off[3], (M - 1) * drs + N) || !fits(1, s.off[2], (M - 1) * srs + K) || !wfits(2, s.off[0], N * K)) return fail("linear: extent");
+            if (!fits(0, s.off[3], (M - 1) * drs + N) || !fits(1, s.off[2], (M - 1) * srs + K) || !wfits(2, s.off[0], (s.n[10] ? 2 : 1) * N * K)) return fail("linear: extent");
+            if (s.n[10] > 1 || (s.n[10] && (s.buf[3] != ZG_NO_BUF || s.n[8] || s.n[9]))) return fail("linear: pairs take no bias and no column range");
+            if (s.n[11] && !s.n[7]) return fail("linear: a row limit needs the rows of a state buffer");
             if (s.buf[3] != ZG_NO_BUF && !wfits(3, s.off[1], N)) return fail("linear: bias extent");
             if (s.buf[0] == s.buf[1]) return fail("linear: in place");
             if (s.n[6] > 6 || (s.n[6] == 5 && !(s.f[0] > 0.0f))) return fail("linear: activation");
@@ -1554,19 +1624,20 @@ bool zg_seq_op_valid(const ZgOp& op, const size_t* elems, size_t n_bufs, char* w
         case ZG_OP_DELTA_RULE: {
             const size_t T = s.n[0], H = s.n[1], G = s.n[2], dim = s.n[3], vdim = s.n[4];
             const size_t form = s.n[10], drs = s.n[11] ? s.n[11] : H * vdim;
-            if (!T || !H || !G || H % G || !dim || !vdim || zg_delta_row_slices((uint32_t)dim) > 32 || form > 31) return fail("delta_rule: shape");
+            if (!T || !H || !G || H % G || !dim || !vdim || zg_delta_row_slices((uint32_t)dim) > 32 || form > 255) return fail("delta_rule: shape");
+            if (((form & 32) && (!(form & 1) || !wfits(5, s.n[14], H * dim))) || (form & 66) == 66) return fail("delta_rule: bonus or decay form");
             if (s.n[12] + H * vdim > drs || ((form & 2) && !(s.f[3] > 0.0f))) return fail("delta_rule: form");
             if (s.off[0] + G * dim > s.n[5] || s.off[1] + G * dim > s.n[5] || s.off[2] + H * vdim > s.n[5] || (!(form & 1) && s.off[3] + H > s.n[6]) || s.n[13] + H * (form & 16 ? 1 : dim) > s.n[7] || s.off[7] + H * vdim > s.n[8])
                 return fail("delta_rule: columns");
             if (!fits(0, 0, (T - 1) * drs + s.n[12] + H * vdim) || !fits(1, 0, T * s.n[5]) || (!(form & 1) && !fits(2, 0, T * s.n[6])) || !fits(3, 0, T * s.n[7]) || !fits(4, 0, T * s.n[8]) ||
-                (!(form & 2) && !wfits(5, s.off[4], H)) || !wfits(5, s.off[5], H * (form & 16 ? 1 : dim)) || !wfits(5, s.off[6], vdim) || !have(6) || elems[s.buf[6]] < H * dim * vdim || !fits(7, 0, ZG_CTL_IDS))
+                (!(form & 66) && !wfits(5, s.off[4], H)) || !wfits(5, s.off[5], H * (form & 16 ? 1 : dim)) || !wfits(5, s.off[6], form & 128 ? H * vdim : vdim) || !have(6) || elems[s.buf[6]] < H * dim * vdim || !fits(7, 0, ZG_CTL_IDS))
                 return fail("delta_rule: extent");
             return true;
         }
         case ZG_OP_ROUTE: {
             const size_t T = s.n[0], NE = s.n[1], top = s.n[2], rs = s.n[3];
-            if (!T || !NE || !top || top > NE || rs < NE || NE > 4096 || s.n[5] > 2) return fail("route: shape");
-            if (s.n[5] == 2 && s.n[6] > 1 && (NE % s.n[6] || s.n[6] > 1024 || !s.n[7] || s.n[7] > s.n[6] || (size_t)s.n[7] * (NE / s.n[6]) < top)) return fail("route: groups");
+            if (!T || !NE || !top || top > NE || rs < NE || NE > 4096 || s.n[5] > 3) return fail("route: shape");
+            if (s.n[5] >= 2 && s.n[6] > 1 && (NE % s.n[6] || s.n[6] > 1024 || !s.n[7] || s.n[7] > s.n[6] || (size_t)s.n[7] * (NE / s.n[6]) < top)) return fail("route: groups");
             if (!fits(0, 0, T * top * 2) || !fits(1, s.off[1], (T - 1) * rs + NE) || !wfits(2, s.off[0], NE)) return fail("route: extent");
             return true;
         }
@@ -1591,6 +1662,7 @@ uint32_t zg_seq_op_writes(uint32_t tag) {
         case ZG_OP_CAUSAL_CONV: return 1u | (1u << 3);
         case ZG_OP_DELTA_RULE: return 1u | (1u << 6);
         case ZG_OP_MOE_FFN: return 1u | (1u << 4);
+        case ZG_OP_STREAM_STEP: return 1u | (1u << 5) | (1u << 6);   // streams, the next sublayer's input, a carried row
         default: return tag >= ZG_OP_SSM_SCAN ? zg_rec_op_writes(tag) : (tag >= ZG_OP_TOKEN_SHIFT ? zg_mix_op_writes(tag) : 1u);
     }
 }
@@ -1606,6 +1678,7 @@ static uint32_t attention_splits(const ZgSeqOp& s) {
     return S < 2 ? 1 : (S > 16 ? 16 : S);
 }
 size_t zg_seq_op_scratch_elems(const ZgOp& op, float* const* bufs) {
+    if (op.tag >= ZG_OP_STREAM_STEP) return 0;
     if (op.tag >= ZG_OP_SSM_SCAN) return zg_rec_op_scratch_elems(op);
     if (op.tag >= ZG_OP_TOKEN_SHIFT) return zg_mix_op_scratch_elems(op);
     if (op.tag == ZG_OP_WINDOW_ATTENTION) {
@@ -1618,7 +1691,7 @@ size_t zg_seq_op_scratch_elems(const ZgOp& op, float* const* bufs) {
     }
     if (!dense_gemm_enabled() || op.tag != ZG_OP_LINEAR || op.u.seq.n[5] != ZG_W_BF16) return 0;
     const ZgSeqOp& s = op.u.seq;
-    if (!zg_dense_gemm_usable(wptr<bf16>(bufs, s.buf[2], s.off[0]), s.n[0], s.n[1], s.n[2])) return 0;
+    if (!zg_dense_gemm_usable(wptr<bf16>(bufs, s.buf[2], s.off[0]), s.n[0], s.n[10] ? 2 * s.n[1] : s.n[1], s.n[2])) return 0;
     return zg_dense_gemm_scratch_elems(s.n[0], s.n[2]);
 }
 
@@ -1628,7 +1701,8 @@ bool zg_launch_seq_op(ZgCudaCtx* ctx, const ZgOp& op, float* const* bufs, float*
     switch (op.tag) {
         case ZG_OP_EMBED:
             ZG_SEQ_WDT(s.n[2], launch_pdl(k_embed<WT>, dim3(s.n[0], (s.n[1] + 255) / 256), dim3(256), 0, st, bufs[s.buf[0]], bufs[s.buf[1]], wptr<WT>(bufs, s.buf[2], s.off[0]), s.n[1], s.f[0],
-                                          s.n[3] ? wptr<WT>(bufs, s.buf[2], s.off[1]) : nullptr, s.n[4] ? wptr<WT>(bufs, s.buf[2], s.off[2]) : nullptr, s.n[4], s.n[5], s.n[6]));
+                                          s.n[3] ? wptr<WT>(bufs, s.buf[2], s.off[1]) : nullptr, s.n[4] ? wptr<WT>(bufs, s.buf[2], s.off[2]) : nullptr, s.n[4], s.n[5], s.n[6],
+                                          s.n[7] ? wptr<WT>(bufs, s.buf[2], s.off[3]) : nullptr));
             ZG_SEQ_CHECK();
             return true;
         case ZG_OP_LINEAR: {
@@ -1636,11 +1710,19 @@ bool zg_launch_seq_op(ZgCudaCtx* ctx, const ZgOp& op, float* const* bufs, float*
             float* dst = bufs[s.buf[0]] + s.off[3];
             const float* src = bufs[s.buf[1]] + s.off[2];
             const bool has_bias = s.buf[3] != ZG_NO_BUF;
+            const bool pairs = s.n[10] != 0;
             const SeqAct act = {s.n[6], s.f[0], s.n[8], s.n[9] ? s.n[9] : N};
             const float* slot_ctl = s.n[7] ? (const float*)bufs[s.buf[4]] : (const float*)nullptr;      // the source is the slot's part of a state buffer
             if (scratch && zg_seq_op_scratch_elems(op, bufs))
                 return zg_dense_gemm_launch(wptr<bf16>(bufs, s.buf[2], s.off[0]), has_bias ? wptr<bf16>(bufs, s.buf[3], s.off[1]) : nullptr, src, dst, M, N, K,
-                                            s.n[3], s.n[4], scratch, st, s.n[6], s.f[0], act.lo, act.hi, slot_ctl, s.n[7]);
+                                            s.n[3], s.n[4], scratch, st, s.n[6], s.f[0], act.lo, act.hi, slot_ctl, s.n[7], pairs, s.n[11]);
+#define ZG_ROWS(PAIRS_)                                                                                                                              \
+    do {                                                                                                                                             \
+        if (vec && M == 1) launch_pdl(k_linear_rows_vec<WT, 1, PAIRS_>, dim3(grid), dim3(256), xs_bytes, st, dst, src, W, b, M, N, K, s.n[3], s.n[4], act, slot_ctl, s.n[7]);      \
+        else if (vec && M <= 4) launch_pdl(k_linear_rows_vec<WT, 4, PAIRS_>, dim3(grid), dim3(256), xs_bytes, st, dst, src, W, b, M, N, K, s.n[3], s.n[4], act, slot_ctl, s.n[7]); \
+        else if (vec) launch_pdl(k_linear_rows_vec<WT, 8, PAIRS_>, dim3(grid), dim3(256), xs_bytes, st, dst, src, W, b, M, N, K, s.n[3], s.n[4], act, slot_ctl, s.n[7]);           \
+        else launch_pdl(k_linear_rows<WT, PAIRS_>, dim3(grid), dim3(256), 0, st, dst, src, W, b, M, N, K, s.n[3], s.n[4], act, slot_ctl, s.n[7]);                                  \
+    } while (0)
             ZG_SEQ_WDT(s.n[5], {
                 const WT* W = wptr<WT>(bufs, s.buf[2], s.off[0]);
                 const WT* b = has_bias ? wptr<WT>(bufs, s.buf[3], s.off[1]) : nullptr;
@@ -1649,15 +1731,15 @@ bool zg_launch_seq_op(ZgCudaCtx* ctx, const ZgOp& op, float* const* bufs, float*
                     const size_t xs_bytes = (size_t)M * K * sizeof(float);
                     const bool vec = K % V == 0 && (reinterpret_cast<size_t>(W) & 15) == 0 && xs_bytes <= 48 * 1024;
                     const dim3 grid((N + 7) / 8);
-                    if (vec && M == 1) launch_pdl(k_linear_rows_vec<WT, 1>, dim3(grid), dim3(256), xs_bytes, st, dst, src, W, b, M, N, K, s.n[3], s.n[4], act, slot_ctl, s.n[7]);
-                    else if (vec && M <= 4) launch_pdl(k_linear_rows_vec<WT, 4>, dim3(grid), dim3(256), xs_bytes, st, dst, src, W, b, M, N, K, s.n[3], s.n[4], act, slot_ctl, s.n[7]);
-                    else if (vec) launch_pdl(k_linear_rows_vec<WT, 8>, dim3(grid), dim3(256), xs_bytes, st, dst, src, W, b, M, N, K, s.n[3], s.n[4], act, slot_ctl, s.n[7]);
-                    else launch_pdl(k_linear_rows<WT>, dim3(grid), dim3(256), 0, st, dst, src, W, b, M, N, K, s.n[3], s.n[4], act, slot_ctl, s.n[7]);
+                    if (pairs) ZG_ROWS(true); else ZG_ROWS(false);
                 } else {
-                    const dim3 grid((N + kTN - 1) / kTN, (M + kTM - 1) / kTM);
-                    k_linear_tile<WT><<<grid, 256, 0, st>>>(dst, src, W, b, M, N, K, s.n[3], s.n[4], act, slot_ctl, s.n[7]);
+                    const uint32_t NW = pairs ? 2 * N : N;
+                    const dim3 grid((NW + kTN - 1) / kTN, (M + kTM - 1) / kTM);
+                    if (pairs) k_linear_tile<WT, true><<<grid, 256, 0, st>>>(dst, src, W, b, M, NW, K, s.n[3], s.n[4], act, slot_ctl, s.n[7], s.n[11]);
+                    else k_linear_tile<WT, false><<<grid, 256, 0, st>>>(dst, src, W, b, M, NW, K, s.n[3], s.n[4], act, slot_ctl, s.n[7], s.n[11]);
                 }
             });
+#undef ZG_ROWS
             ZG_SEQ_CHECK();
             return true;
         }
@@ -1767,19 +1849,20 @@ bool zg_launch_seq_op(ZgCudaCtx* ctx, const ZgOp& op, float* const* bufs, float*
                 const size_t walk_smem = (size_t)2 * kDeltaTile * ((form & kDeltaHeadDecay ? 2 : 3) * dpad + 4) * sizeof(float);
                 ZG_SEQ_WDT(s.n[9], launch_pdl(k_delta_prepare<WT>, dim3((T * H + 3) / 4), dim3(128), 0, st, scratch, bufs[s.buf[1]], betab, bufs[s.buf[3]] + s.n[13],
                                               wptr<WT>(bufs, s.buf[5], 0), T, H, G, dim, dpad, s.off[0], s.off[1], s.off[3], s.off[4], s.off[5], s.n[5], s.n[6], s.n[7], s.f[1], s.f[2],
-                                              form, inv_tau));
+                                              form, inv_tau, s.n[14]));
                 ZG_SEQ_CHECK();
-#define ZG_WALK_FORM(RS_, PLAIN_, HEADG_)                                                                                                       \
+#define ZG_WALK_FORM(RS_, PLAIN_, HEADG_, BONUS_)                                                                                               \
     do {                                                                                                                                        \
-        if (walk_smem > 48 * 1024) cudaFuncSetAttribute(k_delta_walk<RS_, PLAIN_, HEADG_>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)walk_smem); \
-        launch_pdl(k_delta_walk<RS_, PLAIN_, HEADG_>, dim3((vdim + wcols - 1) / wcols, H), dim3(kWalkThreads), walk_smem, st, dst, bufs[s.buf[1]], \
+        if (walk_smem > 48 * 1024) cudaFuncSetAttribute(k_delta_walk<RS_, PLAIN_, HEADG_, BONUS_>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)walk_smem); \
+        launch_pdl(k_delta_walk<RS_, PLAIN_, HEADG_, BONUS_>, dim3((vdim + wcols - 1) / wcols, H), dim3(kWalkThreads), walk_smem, st, dst, bufs[s.buf[1]], \
                    scratch, bufs[s.buf[6]], bufs[s.buf[7]], T, H, dim, vdim, s.off[2], s.n[5], dst_rs);                                         \
     } while (0)
 #define ZG_WALK(RS_)                                                                                                                            \
     case RS_:                                                                                                                                   \
-        if (form & kDeltaPlain) { if (form & kDeltaHeadDecay) ZG_WALK_FORM(RS_, true, true); else ZG_WALK_FORM(RS_, true, false); }             \
-        else if (form & kDeltaHeadDecay) ZG_WALK_FORM(RS_, false, true);                                                                        \
-        else ZG_WALK_FORM(RS_, false, false);                                                                                                   \
+        if (form & kDeltaBonus) { if (form & kDeltaHeadDecay) ZG_WALK_FORM(RS_, true, true, true); else ZG_WALK_FORM(RS_, true, false, true); } \
+        else if (form & kDeltaPlain) { if (form & kDeltaHeadDecay) ZG_WALK_FORM(RS_, true, true, false); else ZG_WALK_FORM(RS_, true, false, false); } \
+        else if (form & kDeltaHeadDecay) ZG_WALK_FORM(RS_, false, true, false);                                                                 \
+        else ZG_WALK_FORM(RS_, false, false, false);                                                                                            \
         break;
                 switch (WS) { ZG_WALK(1) ZG_WALK(2) ZG_WALK(4) ZG_WALK(8) ZG_WALK(16) default: ZG_WALK(32) }
 #undef ZG_WALK
@@ -1788,19 +1871,19 @@ bool zg_launch_seq_op(ZgCudaCtx* ctx, const ZgOp& op, float* const* bufs, float*
                 if (smem > 48 * 1024) cudaFuncSetAttribute(k_delta_rule<WT>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
                 launch_pdl(k_delta_rule<WT>, dim3(grid), dim3(kDeltaThreads), smem, st, dst, bufs[s.buf[1]], betab, bufs[s.buf[3]] + s.n[13], wptr<WT>(bufs, s.buf[5], 0), bufs[s.buf[6]],
                                                                   bufs[s.buf[7]], T, H, G, dim, vdim, RS, s.off[0], s.off[1], s.off[2], s.off[3], s.off[4], s.off[5],
-                                                                  s.n[5], s.n[6], s.n[7], s.f[1], s.f[2], form, inv_tau, dst_rs);
+                                                                  s.n[5], s.n[6], s.n[7], s.f[1], s.f[2], form, inv_tau, dst_rs, s.n[14]);
             });
             ZG_SEQ_CHECK();
             ZG_SEQ_WDT(s.n[9], launch_pdl(k_delta_out<WT>, dim3((T * H + 3) / 4), dim3(128), 0, st, dst, bufs[s.buf[4]] + s.off[7], wptr<WT>(bufs, s.buf[5], 0), T * H, H, vdim, s.n[8], s.off[6], s.f[0],
-                                                           dst_rs, (uint32_t)((form & kDeltaSiluGate) != 0), out_scale));
+                                                           dst_rs, (uint32_t)((form & kDeltaSiluGate) != 0), out_scale, (uint32_t)((form & kDeltaWideNorm) != 0)));
             ZG_SEQ_CHECK();
             return true;
         }
         case ZG_OP_ROUTE: {
             const uint32_t T = s.n[0], NE = s.n[1];
-            const uint32_t groups = s.n[5] == 2 && s.n[6] > 1 ? s.n[6] : 0;
+            const uint32_t groups = s.n[5] >= 2 && s.n[6] > 1 ? s.n[6] : 0;
             ZG_SEQ_WDT(s.n[4], launch_pdl(k_route<WT>, dim3((T + 3) / 4), dim3(128), 4 * (NE + groups) * sizeof(float), st, bufs[s.buf[0]], bufs[s.buf[1]] + s.off[1], wptr<WT>(bufs, s.buf[2], s.off[0]), T, NE,
-                                                                                         s.n[2], s.n[3], s.n[5], groups, s.n[7]));
+                                                                                         s.n[2], s.n[3], s.n[5], groups, s.n[7], s.f[0]));
             ZG_SEQ_CHECK();
             return true;
         }
@@ -1838,6 +1921,7 @@ bool zg_launch_seq_op(ZgCudaCtx* ctx, const ZgOp& op, float* const* bufs, float*
             return true;
         }
         default:
+            if (op.tag >= ZG_OP_STREAM_STEP) return zg_launch_stream_op(op, bufs, st);
             return op.tag >= ZG_OP_SSM_SCAN ? zg_launch_rec_op(op, bufs, scratch, st) : zg_launch_mix_op(op, bufs, scratch, st);
     }
 }

@@ -391,4 +391,15 @@ size_t zg_rec_op_scratch_elems(const ZgOp& op);   // shared scratch of a long SS
 bool zg_launch_rec_op(const ZgOp& op, float* const* bufs, float* scratch, cudaStream_t st);
 size_t zg_seq_op_operand_scratch(const ZgOp& op);   // f32 slots an op's own scratch operand needs (MOE_FFN)
 bool zg_dense_gemm_launch(const void* w_bf16, const void* bias_bf16, const float* src, float* dst, uint32_t M, uint32_t N, uint32_t K,
-                          uint32_t src_rs, uint32_t dst_rs, float* scratch, cudaStream_t st, uint32_t act = 0, float act_p = 0.0f, uint32_t act_lo = 0, uint32_t act_hi = 0xffffffffu, const float* ctl = nullptr, uint32_t slot_stride = 0);   // act: 0 none, 1 + ACTIVATION kind, on columns [act_lo, act_hi)
+                          uint32_t src_rs, uint32_t dst_rs, float* scratch, cudaStream_t st, uint32_t act = 0, float act_p = 0.0f, uint32_t act_lo = 0, uint32_t act_hi = 0xffffffffu, const float* ctl = nullptr, uint32_t slot_stride = 0, bool pairs = false, uint32_t rows_from = 0);
+// act: 0 none, 1 + ACTIVATION kind, on columns [act_lo, act_hi); pairs: W holds 2 N rows, gate and up in turns, dst = act(gate) * up; rows_from > 0 (with ctl): rows
+// from position + rows_from on are not computed.
+// Batched form: head h of `heads` multiplies its own K columns of the source (at h * src_hs) with rows h N .. h N + N - 1 of W (the last head has n_last rows) into
+// columns h * dst_hs of dst; act on the last head's outputs alone.
+bool zg_dense_gemm_batched_usable(uint32_t M, uint32_t N, uint32_t K, uint32_t act);
+size_t zg_dense_gemm_batched_scratch_elems(uint32_t heads, uint32_t M, uint32_t K);
+bool zg_dense_gemm_batched_launch(const void* w_bf16, const float* src, float* dst, uint32_t heads, uint32_t M, uint32_t N, uint32_t n_last, uint32_t K, uint32_t src_hs, uint32_t src_rs,
+                                  uint32_t dst_hs, uint32_t dst_rs, float* scratch, cudaStream_t st, uint32_t act_last, float act_p);
+// streamops.cu : ZG_OP_STREAM_STEP
+bool zg_stream_op_valid(const ZgOp& op, const size_t* elems, size_t n_bufs, char* why, size_t why_n);
+bool zg_launch_stream_op(const ZgOp& op, float* const* bufs, cudaStream_t st);

@@ -51,6 +51,14 @@ def _open_pepevik(be, path, dtype, n_slots, max_chunk, max_tokens):
     return SequenceSession(be, model, n_slots=n_slots, max_chunk=max_chunk, max_context=max_tokens or None)
 
 
+@register("Fomanex")
+def _open_fomanex(be, path, dtype, n_slots, max_chunk, max_tokens):
+    from .fomanex import FomanexModel
+    from .session import SequenceSession
+    model = FomanexModel.load(be, path, dtype)
+    return SequenceSession(be, model, n_slots=n_slots, max_chunk=max_chunk, max_context=max_tokens or None)
+
+
 @register("Fotovik")
 def _open_fotovik(be, path, dtype, n_slots, max_chunk, max_tokens):
     from .fotovik import FotovikModel

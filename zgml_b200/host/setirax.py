@@ -40,6 +40,7 @@ import numpy as np
 
 from .. import abi
 from ..backend import CudaBackend, DeviceBuffer, DeviceOp, DeviceProgram, ExternBuffer
+from .latent import expands
 from .rotary import rotary_frequencies
 from .safetensors import SafetensorsFile
 from .session import LoweredProgram
@@ -50,7 +51,6 @@ ARCHITECTURE = "Setirax"
 DEFAULT_CONTEXT = 4096     # positions a sequence may reach when a layer attends without a window and the caller names no bound
 MIXERS = ("latent_attention", "parallel", "rglru")
 LRU_RATE = 8.0             # log a = -8 r softplus(lam): fixed by the design
-EXPAND_MIN_TOKENS = 128    # steps from this size on expand a latent layer's keys and values per head (bfloat16 sessions)
 
 
 def _tensor_sizes(kind: str, m: dict, mlp: Optional[dict]) -> tuple:
@@ -278,12 +278,8 @@ class SetiraxModel:
         return specs
 
     def _expands(self, T: int, R: int, m: dict) -> bool:
-        """Whether a step of T tokens runs a latent layer in the expanded form.  Expanding costs 2 R rank H (dim + vdim) FLOPs on the
-        tensor cores per step; the absorbed form costs (2 rank - dim - vdim) more multiply-adds per (query, key, head) in f32.  Worth it
-        for long steps of bfloat16 sessions whose latent fits the tensor-core product (rank a multiple of 8, at least 64); float32
-        sessions, whose products are exact f32 tiles either way, and short steps stay absorbed."""
-        rank, per_head = m["kv_rank"], m["dim"] + m["vdim"]
-        return (self.wdt == abi.W_BF16 or self.expand_float32) and T >= EXPAND_MIN_TOKENS and rank % 8 == 0 and rank >= 64 and 2 * rank > per_head
+        """Whether a step of T tokens runs a latent layer in the expanded form."""
+        return expands(T, m["kv_rank"], 0, m["dim"], m["vdim"], self.wdt, self.expand_float32)
 
     # ── lowering ──
     def lower(self, T: int, head: str, pool: SequenceStatePool, keep_layers: bool = False) -> LoweredProgram:
