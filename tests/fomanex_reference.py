@@ -202,4 +202,4 @@ def forward(cfg, p, tokens, return_layers=False):
             X = write_streams(X, p[hc + ".mix"], p[hc + ".out"], m * y)
         sums.append(X.sum(0))
     z = logits_of(dynamic_tanh(X.sum(0), p, "final.norm") @ np.asarray(p["embed"], np.float64).T, cfg)
-    return (z, np.stack(sums)) if return_layers else z
+    return (z, np.array(sums)) if return_layers else z
