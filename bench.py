@@ -773,10 +773,10 @@ def main():
     ap.add_argument("--no-check", action="store_true", help="skip the 2-layer oracle comparison")
     ap.add_argument("--no-cpu", action="store_true")
     ap.add_argument("--no-extras", action="store_true")
-    ap.add_argument("--arch", default="", choices=["", "lududra", "vemepel", "pepevik", "setirax", "fotovik"],
+    ap.add_argument("--arch", default="", choices=["", "lududra", "vemepel", "pepevik", "setirax", "fotovik", "fomanex"],
                     help="side bench instead of the default workload: prefill / decode throughput of that design next to the framework's closest "
-                         "model at equal layer sizes (lududra: a LLaMA; vemepel, pepevik: Lududra; setirax: Pepevik; fotovik: Setirax)")
-    ap.add_argument("--arms", default="", help="--arch pepevik, setirax, fotovik: comma-separated arms to run (default: both)")
+                         "model at equal layer sizes (lududra: a LLaMA; vemepel, pepevik: Lududra; setirax: Pepevik; fotovik: Setirax; fomanex: Setirax, Vemepel)")
+    ap.add_argument("--arms", default="", help="--arch pepevik, setirax, fotovik, fomanex: comma-separated arms to run (default: all)")
     ap.add_argument("--sizes", default="", help="--arch: comma-separated size names (default: all)")
     ap.add_argument("--prefill-tokens", type=int, default=1024, help="--arch: tokens of the timed prefill chunk")
     ap.add_argument("--context", type=int, default=1024, help="--arch: tokens in the sequence before the timed decode steps")

@@ -32,7 +32,7 @@ def vemepel_arm(be, size, prefill_T, context, reps):
     cfgd = synthetic_config(**size)
     cfg = VemepelConfig.from_dict(cfgd)
     model = VemepelModel(be, cfg, synthetic_tensors(cfgd), "bfloat16")
-    s = SequenceSession(be, model, n_slots=1, max_chunk=prefill_T, max_context=context + 64)
+    s = SequenceSession(be, model, n_slots=1, max_chunk=prefill_T, max_context=context + 1024)
     r = np.random.default_rng(0)
     prompt = r.integers(0, cfg.vocab, context).tolist()
     D = cfg.width
